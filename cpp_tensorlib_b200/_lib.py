@@ -89,6 +89,12 @@ SIGNATURES = {
     "tlb_decoder_run": (ci, [vp, i64, vp]),
     "tlb_decoder_step": (ci, [vp, C.POINTER(C.c_int32), C.POINTER(C.c_int32), vp]),
     "tlb_decoder_prefill": (ci, [vp, C.POINTER(C.c_int32), i64, C.POINTER(C.c_int32), vp]),
+    "tlb_decoder_prefill_logits": (ci, [vp, C.POINTER(C.c_int32), i64, C.POINTER(C.c_int32), i64, vp,
+                                        C.POINTER(C.c_int32), vp]),
+    "tlb_stack_create": (ci, [vp, vp, C.POINTER(vp)]),
+    "tlb_stack_set_matrix": (ci, [vp, i64, ci, vp, i64, i64]),
+    "tlb_stack_set_vector": (ci, [vp, i64, ci, ci, vp, i64]),
+    "tlb_stack_state_bytes": (i64, [vp]),
     "tlb_decoder_last_token": (ci, [vp, C.POINTER(C.c_int32), vp]),
     "tlb_decoder_ipc_export": (ci, [vp, vp]),
     "tlb_decoder_ipc_open": (ci, [vp, vp]),

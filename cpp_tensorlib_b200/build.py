@@ -21,13 +21,28 @@ def sources():
     return sorted(glob.glob(os.path.join(CSRC, "*.cu")))
 
 
+def _headers():
+    return glob.glob(os.path.join(CSRC, "*.cuh")) + glob.glob(os.path.join(HERE, "..", "include", "*.h"))
+
+
+def _newer(target, deps):
+    return os.path.exists(target) and all(os.path.getmtime(d) <= os.path.getmtime(target) for d in deps)
+
+
 def _stale():
-    if not os.path.exists(LIB):
-        return True
-    t = os.path.getmtime(LIB)
-    deps = sources() + glob.glob(os.path.join(CSRC, "*.cuh")) + \
-        glob.glob(os.path.join(HERE, "..", "include", "*.h"))
-    return any(os.path.getmtime(d) > t for d in deps)
+    return not _newer(LIB, sources() + _headers())
+
+
+def _includes(path, seen):
+    """The project headers a source reaches through its quoted includes."""
+    with open(path) as f:
+        for line in f:
+            if line.startswith('#include "'):
+                h = os.path.normpath(os.path.join(os.path.dirname(path), line.split('"')[1]))
+                if h not in seen and os.path.exists(h):
+                    seen.add(h)
+                    _includes(h, seen)
+    return seen
 
 
 def build(force=False, verbose=False):
@@ -38,6 +53,8 @@ def build(force=False, verbose=False):
     for src in sources():
         obj = src[:-3] + ".o"
         objs.append(obj)
+        if not (force or verbose) and _newer(obj, [src] + sorted(_includes(src, set()))):
+            continue
         cmd = [NVCC] + FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-c", src, "-o", obj]
         procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT)))
     for src, p in procs:

@@ -21,6 +21,7 @@
 #include <vector>
 
 #include "comm.cuh"
+#include "decoder_base.cuh"
 #include "gemv_q4p.cuh"
 
 namespace tlb {
@@ -85,9 +86,9 @@ struct DecLayer {
   float *Kc = nullptr, *Vc = nullptr;
 };
 
-struct Decoder {
+struct Decoder : DecoderBase {
   // sizes local to this rank (hidden and vocab_offset are global notions)
-  int hidden = 0, n_layers = 0, n_q = 0, n_kv = 0, hd = 0, ff = 0, vocab = 0, max_ctx = 0;
+  int n_layers = 0, n_q = 0, n_kv = 0, hd = 0, ff = 0;
   float eps = 1e-6f, rope_base = 1e6f, scale = 1.f;
   int tp_rank = 0, tp_size = 1;
   int kv_bf16 = 0;   // caches hold bf16 (kv_cache::init with dtype::bf16, include/cuda.h:1336-1346)
@@ -97,13 +98,9 @@ struct Decoder {
   const float *embed = nullptr, *onorm = nullptr;
   // scratch
   float *x = nullptr, *xb = nullptr, *hb = nullptr, *qkv = nullptr, *att = nullptr, *t0 = nullptr,
-        *t1 = nullptr, *gu = nullptr, *mb = nullptr, *logits = nullptr;
+        *t1 = nullptr, *gu = nullptr, *mb = nullptr;
   void* attn_partials = nullptr;
-  unsigned* d_pos = nullptr;
   float2* rope_cs = nullptr;  // [hd/2] (cos, sin) of the current position, refreshed per token
-  int* d_tok = nullptr;      // token consumed by the next forward; overwritten with the result
-  int* d_tok_out = nullptr;  // copy of the last result (read back by the host)
-  int *h_tok = nullptr, *h_out = nullptr;  // pinned
   // tensor-parallel exchange
   CommDev comm;
   uint2* stage_local = nullptr;
@@ -112,35 +109,19 @@ struct Decoder {
   void* peer_flags_base[TP_MAX] = {};
   bool peers_open = false;
   void* sink[TP_MAX] = {};          // loopback drill: stand-ins for peers that never answer
-  // batched prompt pass: row-batched scratch for chunks of up to PF_CHUNK tokens
+  // batched prompt pass: row-batched scratch, carved from one allocation of pf_rows rows
   float* pf = nullptr;
-  int* pf_ids = nullptr;
-  int pf_rows = 0;          // rows the prefill scratch was sized for
-  // graph
-  cudaGraphExec_t graph = nullptr;
-  long long launches_per_token = 0;
-  // Host mirror of the device-resident position (captured_decoder::cur_pos of the reference,
-  // bench/cuda/qwen_model.h:877-885): every entry point that advances the sequence checks it
-  // against the cache capacity before anything is launched.
-  long long host_pos = 0;
-  long long vocab_total = 0;   // rows of the embedding table (0: unknown, ids are only checked >= 0)
-};
+  int pf_rows = 0;
+  float *pf_res[2] = {}, *pf_h = nullptr, *pf_h2 = nullptr, *pf_md = nullptr, *pf_qkv = nullptr, *pf_qkvh = nullptr,
+        *pf_ah = nullptr, *pf_at = nullptr, *pf_gu = nullptr, *pf_mb = nullptr;
 
-// The reference's feed() returns false when cur_pos >= max_ctx (bench/cuda/qwen_model.h:879);
-// here the refusal is an argument error and nothing is launched.
-static int room_for(Decoder* d, long long n, const char* who) {
-  if (d->host_pos + n > d->max_ctx)
-    return set_error(TLB_ERR_ARG, std::string(who) + ": position " + std::to_string(d->host_pos) + " + " +
-                                      std::to_string(n) + " token(s) exceeds the cache capacity " +
-                                      std::to_string(d->max_ctx));
-  return TLB_OK;
-}
-static int token_ok(Decoder* d, long long token, const char* who) {
-  if (token < 0 || (d->vocab_total > 0 && token >= d->vocab_total))
-    return set_error(TLB_ERR_ARG, std::string(who) + ": token id " + std::to_string(token) +
-                                      " outside the embedding table");
-  return TLB_OK;
-}
+  ~Decoder() override;
+  int forward(cudaStream_t s) override;
+  int prefill_rows() const override { return prefill_chunk_rows(1024); }
+  int prefill_begin(int rows, cudaStream_t s) override;
+  int prefill_pass(const int* d_ids, int rows, int pos, cudaStream_t s) override;
+  int head_rows(const int* rows, int n, float* out, cudaStream_t s) override;
+};
 
 static int set_linear(Linear& L, const void* q4, int K, int N, int pair_h = 0) {
   L.q4 = q4;
@@ -222,7 +203,8 @@ static PairEpi swiglu_epilogue(const Decoder* d) {
 }
 
 
-static int forward(Decoder* d, cudaStream_t s) {
+int Decoder::forward(cudaStream_t s) {
+  Decoder* d = this;
   DeviceCtx* c = nullptr;
   int rc = get_ctx(&c);
   if (rc) return rc;
@@ -417,9 +399,117 @@ static int forward(Decoder* d, cudaStream_t s) {
   return TLB_OK;
 }
 
+Decoder::~Decoder() {
+  if (peers_open)
+    for (int r = 0; r < tp_size; r++)
+      if (r != tp_rank) {
+        if (peer_stage_base[r]) cudaIpcCloseMemHandle(peer_stage_base[r]);
+        if (peer_flags_base[r]) cudaIpcCloseMemHandle(peer_flags_base[r]);
+      }
+  for (auto& L : layers) {
+    cudaFree(L.Kc); cudaFree(L.Vc);
+    cudaFree(L.wqkv.packed); cudaFree(L.wo.packed); cudaFree(L.wgu.packed); cudaFree(L.wd.packed);
+  }
+  cudaFree(lm_head.packed);
+  float* bufs[] = {x, xb, t1, hb, qkv, att, t0, gu, mb};
+  for (float* b : bufs) cudaFree(b);
+  cudaFree(stage_local);
+  for (void* sk : sink) cudaFree(sk);
+  cudaFree(rope_cs);
+  cudaFree(pf);
+  cudaFree(attn_partials); cudaFree(flags_local);
+}
+
+// ---- batched prompt pass (bench/cuda/qwen_model.h:357-442 prefill_chunk_ / prefill_batched):
+// the same forward as the decode step with one row per prompt token -- every projection is a
+// GEMM on the int4 weights (tensor cores for more than 8 rows), attention is one tiled causal
+// pass over the cache.  Single GPU; the weights are read in the reference layout the caller
+// handed to tlb_decoder_set_linear, which must still be alive.
+int Decoder::prefill_begin(int rows, cudaStream_t s) {
+  if (tp_size != 1) return set_error(TLB_ERR_UNSUPPORTED, "tlb_decoder_prefill: single GPU only");
+  if (!embed || !onorm) return set_error(TLB_ERR_STATE, "decoder: embed / final norm not set");
+  if (pf && pf_rows >= rows) return TLB_OK;
+  const int E = hidden, D = hd, QKV = (n_q + 2 * n_kv) * D;
+  const size_t CH = rows, n_emb = CH * E, n_qkv = CH * QKV, n_att = CH * n_q * D, n_gu = CH * 2 * ff, n_mb = CH * ff;
+  const size_t total = 5 * n_emb /* res0 res1 h h2 md */ + 2 * n_qkv + 2 * n_att + n_gu + n_mb;
+  if (pf) {
+    TLB_CUDA(cudaStreamSynchronize(s));
+    TLB_CUDA(cudaFree(pf));
+    pf = nullptr;
+  }
+  TLB_CUDA(cudaMalloc(&pf, total * sizeof(float)));
+  pf_rows = rows;
+  float* p = pf;
+  auto take = [&](size_t n) { float* r = p; p += n; return r; };
+  pf_res[0] = take(n_emb); pf_res[1] = take(n_emb);
+  pf_h = take(n_emb); pf_h2 = take(n_emb); pf_md = take(n_emb);
+  pf_qkv = take(n_qkv); pf_qkvh = take(n_qkv);
+  pf_ah = take(n_att); pf_at = take(n_att);
+  pf_gu = take(n_gu); pf_mb = take(n_mb);
+  return TLB_OK;
+}
+
+int Decoder::prefill_pass(const int* d_ids, int rows, int pos, cudaStream_t s) {
+  DeviceCtx* c = nullptr;
+  int rc = get_ctx(&c);
+  if (rc) return rc;
+  const int E = hidden, D = hd, NQ = n_q, NKV = n_kv, FF = ff;
+  const int QKV = (NQ + 2 * NKV) * D;
+  float *hrow = pf_h, *h2 = pf_h2, *md = pf_md, *qkv = pf_qkv, *qkvh = pf_qkvh, *ah = pf_ah, *at = pf_at, *gu = pf_gu,
+        *mb = pf_mb;
+  auto gemm = [&](const Linear& L, const float* x, float* y, int rows) -> int {
+    if (!L.q4) return set_error(TLB_ERR_STATE, "decoder: a linear weight was never set");
+    return tlb_gemm_q4(x, rows, L.K, L.q4, L.scales(), y, L.N, L.N, L.K, 1.0f, 0.0f, s);
+  };
+#define PF(expr) do { rc = (expr); if (rc) return rc; } while (0)
+  float* x = pf_res[1];   // the chunk's embeddings; layer l writes its residual into pf_res[l & 1]
+  PF(launch_embed_rows(embed, d_ids, x, E, rows, s));
+  PF(launch_rmsnorm(x, layers[0].an, hrow, E, eps, rows, s));
+  for (int l = 0; l < n_layers; l++) {
+    DecLayer& L = layers[l];
+    float* ro = pf_res[l & 1];
+    PF(gemm(L.wqkv, hrow, qkv, rows));
+    // token-major [rows, q|k|v] -> head-major [n_q + 2 n_kv, rows, D], biases riding along
+    float* kh = qkvh + (size_t)NQ * rows * D;
+    float* vh = qkvh + (size_t)(NQ + NKV) * rows * D;
+    PF(launch_split_heads(qkv, L.bq, qkvh, rows, QKV, 0, NQ, D, s));
+    PF(launch_split_heads(qkv, L.bk, kh, rows, QKV, (long long)NQ * D, NKV, D, s));
+    PF(launch_split_heads(qkv, L.bv, vh, rows, QKV, (long long)(NQ + NKV) * D, NKV, D, s));
+    // [H, rows, D] flattened: row r = h*rows + t, so rope's position is pos + r % rows
+    PF(launch_rope(qkvh, nullptr, qkvh, NQ * rows, rows, D, (unsigned)pos, nullptr, rope_base, s));
+    PF(launch_rope(kh, nullptr, kh, NKV * rows, rows, D, (unsigned)pos, nullptr, rope_base, s));
+    PF(launch_kv_fill(L.Kc, L.Vc, kh, vh, rows, max_ctx, NKV, D, pos, kv_bf16, s));
+    PF(launch_attn_prefill(c, qkvh, L.Kc, L.Vc, ah, NQ, NKV, rows, max_ctx, D, scale, pos,
+                           kv_bf16, s));
+    PF(launch_merge_heads(ah, at, rows, NQ, D, s));
+    PF(gemm(L.wo, at, md, rows));
+    PF(launch_add_rmsnorm(x, md, L.fn, ro, h2, E, eps, rows, s));
+    PF(gemm(L.wgu, h2, gu, rows));
+    PF(launch_swiglu(gu, mb, FF, rows, s));
+    PF(gemm(L.wd, mb, md, rows));
+    const float* nextw = (l + 1 < n_layers) ? layers[l + 1].an : onorm;
+    PF(launch_add_rmsnorm(ro, md, nextw, ro, hrow, E, eps, rows, s));
+    x = ro;
+  }
+#undef PF
+  return TLB_OK;
+}
+
+// hrow of the pass holds the final norm of every row
+int Decoder::head_rows(const int* rows, int n, float* out, cudaStream_t s) {
+  DeviceCtx* c = nullptr;
+  int rc = get_ctx(&c);
+  for (int i = 0; i < n && !rc; i++)
+    rc = run_linear(c, lm_head, pf_h + (size_t)rows[i] * hidden, out + (size_t)i * vocab, s, nullptr);
+  return rc;
+}
+
 }  // namespace tlb
 
 using namespace tlb;
+
+// the handle as this model, NULL when it is another one's
+static Decoder* as_q4(void* h) { return dynamic_cast<Decoder*>((DecoderBase*)h); }
 
 extern "C" {
 
@@ -464,18 +554,12 @@ int tlb_decoder_create(const int64_t* cfg, int n_cfg, float eps, float rope_base
   TLB_CUDA(fa(&d->t0, d->hidden));
   TLB_CUDA(fa(&d->gu, (size_t)2 * d->ff));
   TLB_CUDA(fa(&d->mb, d->ff));
-  TLB_CUDA(fa(&d->logits, d->vocab));
   size_t pb = 256 + attn_partials_bytes(d->n_q, d->n_kv, d->max_ctx, d->hd, c->sm_count);
   TLB_CUDA(cudaMalloc(&d->attn_partials, pb));
   TLB_CUDA(cudaMemset(d->attn_partials, 0, pb));
   TLB_CUDA(cudaMalloc(&d->rope_cs, (size_t)(d->hd / 2) * sizeof(float2)));
-  TLB_CUDA(cudaMalloc(&d->d_pos, 16));
-  TLB_CUDA(cudaMemset(d->d_pos, 0, 16));
-  TLB_CUDA(cudaMalloc(&d->d_tok, 16));
-  TLB_CUDA(cudaMemset(d->d_tok, 0, 16));
-  d->d_tok_out = d->d_tok + 1;
-  TLB_CUDA(cudaMallocHost(&d->h_tok, 64));
-  d->h_out = d->h_tok + 4;
+  rc = d->init_base();
+  if (rc) return rc;
   // exchange buffers (allocated even at tp_size 1: tiny)
   d->comm.rank = d->tp_rank;
   d->comm.size = d->tp_size;
@@ -488,35 +572,7 @@ int tlb_decoder_create(const int64_t* cfg, int n_cfg, float eps, float rope_base
   d->comm.stage[d->tp_rank] = d->stage_local;
   d->comm.seq = d->flags_local;
   TLB_CUDA(cudaDeviceSynchronize());
-  *out = d;
-  return TLB_OK;
-}
-
-int tlb_decoder_destroy(void* h) {
-  auto* d = (Decoder*)h;
-  if (!d) return TLB_OK;
-  cudaDeviceSynchronize();
-  if (d->graph) cudaGraphExecDestroy(d->graph);
-  if (d->peers_open)
-    for (int r = 0; r < d->tp_size; r++)
-      if (r != d->tp_rank) {
-        if (d->peer_stage_base[r]) cudaIpcCloseMemHandle(d->peer_stage_base[r]);
-        if (d->peer_flags_base[r]) cudaIpcCloseMemHandle(d->peer_flags_base[r]);
-      }
-  for (auto& L : d->layers) {
-    cudaFree(L.Kc); cudaFree(L.Vc);
-    cudaFree(L.wqkv.packed); cudaFree(L.wo.packed); cudaFree(L.wgu.packed); cudaFree(L.wd.packed);
-  }
-  cudaFree(d->lm_head.packed);
-  float* bufs[] = {d->x, d->xb, d->t1, d->hb, d->qkv, d->att, d->t0, d->gu, d->mb, d->logits};
-  for (float* b : bufs) cudaFree(b);
-  cudaFree(d->stage_local);
-  for (void* sk : d->sink) cudaFree(sk);
-  cudaFree(d->rope_cs);
-  cudaFree(d->pf); cudaFree(d->pf_ids);
-  cudaFree(d->attn_partials); cudaFree(d->d_pos); cudaFree(d->d_tok); cudaFree(d->flags_local);
-  cudaFreeHost(d->h_tok);
-  delete d;
+  *out = static_cast<DecoderBase*>(d);
   return TLB_OK;
 }
 
@@ -524,7 +580,7 @@ int tlb_decoder_destroy(void* h) {
 //        3 wd [ff -> hidden]  4 lm_head [hidden -> vocab] (layer ignored).
 // q4 is a DEVICE pointer to a buffer in the q4 layout, borrowed for the decoder's life.
 int tlb_decoder_set_linear(void* h, int64_t layer, int which, const void* q4, int64_t K, int64_t N) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d && q4 && K > 0 && N > 0 && K % 32 == 0, "tlb_decoder_set_linear: bad arguments");
   const int E = d->hidden, QKV = (d->n_q + 2 * d->n_kv) * d->hd;
   Linear* L = nullptr;
@@ -549,7 +605,7 @@ int tlb_decoder_set_linear(void* h, int64_t layer, int which, const void* q4, in
 // which: 0 attn norm  1 ffn norm  2 bq  3 bk  4 bv (may be NULL: no bias)  5 final norm
 //        6 embedding table [vocab_total, hidden] (layer ignored for 5 and 6). Device pointers.
 int tlb_decoder_set_vector(void* h, int64_t layer, int which, const float* v) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d, "tlb_decoder_set_vector: null decoder");
   if (which == 5) { d->onorm = v; return TLB_OK; }
   if (which == 6) { d->embed = v; return TLB_OK; }
@@ -564,246 +620,16 @@ int tlb_decoder_set_vector(void* h, int64_t layer, int which, const float* v) {
 // Device pointers of one layer's K and V cache ([n_kv, max_ctx, hd] f32) so the
 // caller can pre-fill a context.
 int tlb_decoder_kv(void* h, int64_t layer, void** K, void** V) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d && K && V && layer >= 0 && layer < d->n_layers, "tlb_decoder_kv: bad arguments");
   *K = d->layers[layer].Kc;
   *V = d->layers[layer].Vc;
   return TLB_OK;
 }
-int tlb_decoder_logits(void* h, void** logits) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && logits, "tlb_decoder_logits: bad arguments");
-  *logits = d->logits;
-  return TLB_OK;
-}
-int tlb_decoder_set_pos(void* h, int64_t pos, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && pos >= 0 && pos < d->max_ctx, "tlb_decoder_set_pos: position outside the cache");
-  d->h_tok[8] = (int)pos;
-  TLB_CUDA(cudaMemcpyAsync(d->d_pos, &d->h_tok[8], 4, cudaMemcpyHostToDevice, (cudaStream_t)stream));
-  TLB_CUDA(cudaStreamSynchronize((cudaStream_t)stream));
-  d->host_pos = pos;
-  return TLB_OK;
-}
-int tlb_decoder_set_token(void* h, int64_t token, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d, "tlb_decoder_set_token: null decoder");
-  {
-    const int rc = token_ok(d, token, "tlb_decoder_set_token");
-    if (rc) return rc;
-  }
-  d->h_tok[0] = (int)token;
-  TLB_CUDA(cudaMemcpyAsync(d->d_tok, d->h_tok, 4, cudaMemcpyHostToDevice, (cudaStream_t)stream));
-  TLB_CUDA(cudaStreamSynchronize((cudaStream_t)stream));
-  return TLB_OK;
-}
-
-
-// Enqueue one token's launches on `stream` (capturable: no sync, no allocation).
-int tlb_decoder_forward(void* h, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d, "tlb_decoder_forward: null decoder");
-  int rc = room_for(d, 1, "tlb_decoder_forward");
-  if (rc) return rc;
-  rc = forward(d, (cudaStream_t)stream);
-  if (!rc) d->host_pos++;
-  return rc;
-}
-int64_t tlb_decoder_launches_per_token(void* h) {
-  auto* d = (Decoder*)h;
-  return d ? d->launches_per_token : 0;
-}
-
-// Capture one forward into an executable graph owned by the decoder
-// (qwen_model.h:791-905 captured_decoder::init_).
-int tlb_decoder_capture(void* h) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d, "tlb_decoder_capture: null decoder");
-  if (d->graph) { cudaGraphExecDestroy(d->graph); d->graph = nullptr; }
-  cudaStream_t s;
-  TLB_CUDA(cudaStreamCreateWithFlags(&s, cudaStreamNonBlocking));
-  TLB_CUDA(cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal));
-  int rc = forward(d, s);
-  cudaGraph_t g = nullptr;
-  cudaError_t e = cudaStreamEndCapture(s, &g);
-  cudaStreamDestroy(s);
-  if (rc) { if (g) cudaGraphDestroy(g); return rc; }
-  if (e != cudaSuccess) return cuda_fail(e, "cudaStreamEndCapture");
-  e = cudaGraphInstantiate(&d->graph, g, 0);
-  cudaGraphDestroy(g);
-  if (e != cudaSuccess) return cuda_fail(e, "cudaGraphInstantiate");
-  return TLB_OK;
-}
-
-// Replay the captured token `n` times back to back; the token id feeds back on
-// the device (greedy decoding with no host round trip).
-int tlb_decoder_run(void* h, int64_t n, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && d->graph, "tlb_decoder_run: capture the decoder first");
-  TLB_REQUIRE(n >= 0, "tlb_decoder_run: negative token count");
-  const int rc = room_for(d, n, "tlb_decoder_run");
-  if (rc) return rc;
-  for (int64_t i = 0; i < n; i++) {
-    TLB_CUDA(cudaGraphLaunch(d->graph, (cudaStream_t)stream));
-    d->host_pos++;
-  }
-  return TLB_OK;
-}
-
-// End-to-end step with HOST buffers: token id in (host), next token id out (host).
-// H2D of the id, one graph replay (or eager launches when not captured), D2H of
-// the result, stream synchronised.  token_in < 0 keeps the device-resident token.
-int tlb_decoder_step(void* h, const int32_t* token_in, int32_t* token_out, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && token_out, "tlb_decoder_step: bad arguments");
-  cudaStream_t s = (cudaStream_t)stream;
-  {
-    int rc = room_for(d, 1, "tlb_decoder_step");
-    if (!rc && token_in && *token_in >= 0) rc = token_ok(d, *token_in, "tlb_decoder_step");
-    if (rc) return rc;
-  }
-  if (token_in && *token_in >= 0) {
-    d->h_tok[0] = *token_in;
-    TLB_CUDA(cudaMemcpyAsync(d->d_tok, d->h_tok, 4, cudaMemcpyHostToDevice, s));
-  }
-  if (d->graph) TLB_CUDA(cudaGraphLaunch(d->graph, s));
-  else {
-    int rc = forward(d, s);
-    if (rc) return rc;
-  }
-  d->host_pos++;
-  TLB_CUDA(cudaMemcpyAsync(d->h_out, d->d_tok_out, 4, cudaMemcpyDeviceToHost, s));
-  TLB_CUDA(cudaStreamSynchronize(s));
-  *token_out = d->h_out[0];
-  return TLB_OK;
-}
-// ---- batched prompt pass (bench/cuda/qwen_model.h:357-442 prefill_chunk_ / prefill_batched):
-// the same forward as the decode step with one row per prompt token -- every projection is a
-// GEMM on the int4 weights (tensor cores for more than 8 rows), attention is one tiled causal
-// pass over the cache -- in chunks of up to 1024 tokens starting at the decoder's current
-// position.  Leaves the caches and the position at pos + T, the greedy next token in the
-// device-resident token cell (so tlb_decoder_run continues from there) and in *next_token.
-// Single GPU; the weights are read in the reference layout the caller handed to
-// tlb_decoder_set_linear, which must still be alive.
-int tlb_decoder_prefill(void* h, const int32_t* tokens, int64_t T, int32_t* next_token, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && tokens && T > 0, "tlb_decoder_prefill: bad arguments");
-  if (d->tp_size != 1) return set_error(TLB_ERR_UNSUPPORTED, "tlb_decoder_prefill: single GPU only");
-  if (!d->embed || !d->onorm) return set_error(TLB_ERR_STATE, "decoder: embed / final norm not set");
-  DeviceCtx* c = nullptr;
-  int rc = get_ctx(&c);
-  if (rc) return rc;
-  cudaStream_t s = (cudaStream_t)stream;
-  // rows per pass: enough CTAs for the narrow (hidden-wide) projections; TLB_PREFILL_CHUNK overrides
-  int CH = 1024;
-  if (const char* e = getenv("TLB_PREFILL_CHUNK")) CH = atoi(e) < 16 ? 16 : (atoi(e) > 8192 ? 8192 : atoi(e));
-  const int E = d->hidden, D = d->hd, NQ = d->n_q, NKV = d->n_kv, FF = d->ff;
-  const int QKV = (NQ + 2 * NKV) * D;
-  unsigned pos0 = 0;
-  TLB_CUDA(cudaMemcpyAsync(&pos0, d->d_pos, 4, cudaMemcpyDeviceToHost, s));
-  TLB_CUDA(cudaStreamSynchronize(s));
-  if ((long long)pos0 + T > d->max_ctx)
-    return set_error(TLB_ERR_ARG, "tlb_decoder_prefill: the prompt does not fit the cache");
-  for (int64_t i = 0; i < T; i++) {
-    rc = token_ok(d, tokens[i], "tlb_decoder_prefill");
-    if (rc) return rc;
-  }
-  // row-batched scratch, carved from one allocation
-  const size_t n_emb = (size_t)CH * E, n_qkv = (size_t)CH * QKV, n_att = (size_t)CH * NQ * D,
-               n_gu = (size_t)CH * 2 * FF, n_mb = (size_t)CH * FF;
-  const size_t total = 5 * n_emb /* res0 res1 h h2 md */ + 2 * n_qkv + 2 * n_att + n_gu + n_mb;
-  if (d->pf && d->pf_rows < CH) {
-    TLB_CUDA(cudaStreamSynchronize(s));
-    TLB_CUDA(cudaFree(d->pf));
-    TLB_CUDA(cudaFree(d->pf_ids));
-    d->pf = nullptr;
-    d->pf_ids = nullptr;
-  }
-  if (!d->pf) {
-    TLB_CUDA(cudaMalloc(&d->pf, total * sizeof(float)));
-    TLB_CUDA(cudaMalloc(&d->pf_ids, CH * sizeof(int)));
-    d->pf_rows = CH;
-  }
-  float* p = d->pf;
-  float* res[2] = {p, p + n_emb};
-  p += 2 * n_emb;
-  float* hrow = p; p += n_emb;
-  float* h2 = p; p += n_emb;
-  float* md = p; p += n_emb;
-  float* qkv = p; p += n_qkv;
-  float* qkvh = p; p += n_qkv;
-  float* ah = p; p += n_att;
-  float* at = p; p += n_att;
-  float* gu = p; p += n_gu;
-  float* mb = p;
-  auto gemm = [&](const Linear& L, const float* x, float* y, int rows) -> int {
-    if (!L.q4) return set_error(TLB_ERR_STATE, "decoder: a linear weight was never set");
-    return tlb_gemm_q4(x, rows, L.K, L.q4, L.scales(), y, L.N, L.N, L.K, 1.0f, 0.0f, s);
-  };
-#define PF(expr) do { rc = (expr); if (rc) return rc; } while (0)
-  int last_rows = 0;
-  for (int64_t t0 = 0; t0 < T; t0 += CH) {
-    const int rows = (int)((T - t0) < CH ? (T - t0) : CH);
-    const unsigned pos = pos0 + (unsigned)t0;
-    last_rows = rows;
-    TLB_CUDA(cudaMemcpyAsync(d->pf_ids, tokens + t0, (size_t)rows * sizeof(int), cudaMemcpyHostToDevice, s));
-    float* x = res[1];   // the chunk's embeddings; layer l writes its residual into res[l & 1]
-    PF(launch_embed_rows(d->embed, d->pf_ids, x, E, rows, s));
-    PF(launch_rmsnorm(x, d->layers[0].an, hrow, E, d->eps, rows, s));
-    for (int l = 0; l < d->n_layers; l++) {
-      DecLayer& L = d->layers[l];
-      float* ro = res[l & 1];
-      PF(gemm(L.wqkv, hrow, qkv, rows));
-      // token-major [rows, q|k|v] -> head-major [n_q + 2 n_kv, rows, D], biases riding along
-      float* kh = qkvh + (size_t)NQ * rows * D;
-      float* vh = qkvh + (size_t)(NQ + NKV) * rows * D;
-      PF(launch_split_heads(qkv, L.bq, qkvh, rows, QKV, 0, NQ, D, s));
-      PF(launch_split_heads(qkv, L.bk, kh, rows, QKV, (long long)NQ * D, NKV, D, s));
-      PF(launch_split_heads(qkv, L.bv, vh, rows, QKV, (long long)(NQ + NKV) * D, NKV, D, s));
-      // [H, rows, D] flattened: row r = h*rows + t, so rope's position is pos + r % rows
-      PF(launch_rope(qkvh, nullptr, qkvh, NQ * rows, rows, D, pos, nullptr, d->rope_base, s));
-      PF(launch_rope(kh, nullptr, kh, NKV * rows, rows, D, pos, nullptr, d->rope_base, s));
-      PF(launch_kv_fill(L.Kc, L.Vc, kh, vh, rows, d->max_ctx, NKV, D, (int)pos, d->kv_bf16, s));
-      PF(launch_attn_prefill(c, qkvh, L.Kc, L.Vc, ah, NQ, NKV, rows, d->max_ctx, D, d->scale, (int)pos,
-                             d->kv_bf16, s));
-      PF(launch_merge_heads(ah, at, rows, NQ, D, s));
-      PF(gemm(L.wo, at, md, rows));
-      PF(launch_add_rmsnorm(x, md, L.fn, ro, h2, E, d->eps, rows, s));
-      PF(gemm(L.wgu, h2, gu, rows));
-      PF(launch_swiglu(gu, mb, FF, rows, s));
-      PF(gemm(L.wd, mb, md, rows));
-      const float* nextw = (l + 1 < d->n_layers) ? d->layers[l + 1].an : d->onorm;
-      PF(launch_add_rmsnorm(ro, md, nextw, ro, hrow, E, d->eps, rows, s));
-      x = ro;
-    }
-  }
-  // logits only for the last row of the last chunk (hrow holds its final norm)
-  PF(run_linear(c, d->lm_head, hrow + (size_t)(last_rows - 1) * E, d->logits, s, nullptr));
-  PF(launch_argmax(c, d->logits, d->vocab, d->d_tok, d->d_tok_out, s));
-#undef PF
-  const unsigned newpos = pos0 + (unsigned)T;
-  d->h_tok[1] = (int)newpos;
-  TLB_CUDA(cudaMemcpyAsync(d->d_pos, &d->h_tok[1], 4, cudaMemcpyHostToDevice, s));
-  TLB_CUDA(cudaMemcpyAsync(d->h_out, d->d_tok_out, 4, cudaMemcpyDeviceToHost, s));
-  TLB_CUDA(cudaStreamSynchronize(s));
-  d->host_pos = (long long)newpos;
-  if (next_token) *next_token = d->h_out[0];
-  return TLB_OK;
-}
-
-int tlb_decoder_last_token(void* h, int32_t* token_out, void* stream) {
-  auto* d = (Decoder*)h;
-  TLB_REQUIRE(d && token_out, "tlb_decoder_last_token: bad arguments");
-  TLB_CUDA(cudaMemcpyAsync(d->h_out, d->d_tok_out, 4, cudaMemcpyDeviceToHost, (cudaStream_t)stream));
-  TLB_CUDA(cudaStreamSynchronize((cudaStream_t)stream));
-  *token_out = d->h_out[0];
-  return TLB_OK;
-}
-
 // ---- tensor-parallel wiring: exchange 128-byte records between the ranks (any
 // host channel), then open the peers' buffers.  Record = two CUDA IPC handles.
 int tlb_decoder_ipc_export(void* h, void* record128) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d && record128, "tlb_decoder_ipc_export: bad arguments");
   cudaIpcMemHandle_t a, b;
   TLB_CUDA(cudaIpcGetMemHandle(&a, d->stage_local));
@@ -814,7 +640,7 @@ int tlb_decoder_ipc_export(void* h, void* record128) {
 }
 // records: tp_size consecutive 128-byte records, index = rank.
 int tlb_decoder_ipc_open(void* h, const void* records) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d && records, "tlb_decoder_ipc_open: bad arguments");
   for (int r = 0; r < d->tp_size; r++) {
     if (r == d->tp_rank) continue;
@@ -835,7 +661,7 @@ int tlb_decoder_ipc_open(void* h, const void* records) {
 // polls for: its next exchange runs into the bounded wait, the kernels return, and
 // tlb_device_status reports TLB_ERR_DEVICE_WAIT.  Nothing faults or hangs.
 int tlb_decoder_loopback_peers(void* h) {
-  auto* d = (Decoder*)h;
+  auto* d = as_q4(h);
   TLB_REQUIRE(d, "tlb_decoder_loopback_peers: null decoder");
   if (d->peers_open) return set_error(TLB_ERR_STATE, "tlb_decoder_loopback_peers: real peers are open already");
   const size_t sb = (size_t)2 * d->tp_size * d->comm.slot_floats * sizeof(uint2);

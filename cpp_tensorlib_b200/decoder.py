@@ -15,6 +15,7 @@ import torch
 
 from ._lib import TlbError, check, lib
 from .cuda import Q4Weight, q4_bytes, to_q4
+from .sequence import Sequence
 
 LINEAR = dict(wqkv=0, wo=1, wgu=2, wd=3, lm_head=4)
 VECTOR = dict(an=0, fn=1, bq=2, bk=3, bv=4, onorm=5, embed=6)
@@ -146,7 +147,7 @@ def host_barrier(store, name, rank, world, timeout_s=60.0, poll_s=0.01):
         time.sleep(poll_s)
 
 
-class Q4Decoder:
+class Q4Decoder(Sequence):
     """Handle on the native decoder.  Weights are device tensors kept alive here
     (the native side borrows their pointers)."""
 
@@ -162,10 +163,9 @@ class Q4Decoder:
         arr = (C.c_int64 * 13)(cfg["hidden"], cfg["layers"], p["n_q"], p["n_kv"], cfg["hd"],
                                p["ff_local"], p["vocab_local"], max_ctx, tp_rank, tp_size,
                                p["vocab"][0], cfg["vocab"], 1 if self.kv_bf16 else 0)
-        self.h = C.c_void_p()
+        super().__init__(p["vocab_local"], max_ctx)
         check(lib().tlb_decoder_create(arr, 13, cfg["eps"], cfg["rope_base"], C.byref(self.h)))
         self._keep = {}
-        self.captured = False
 
     def _stream(self):
         return C.c_void_p(torch.cuda.current_stream().cuda_stream)
@@ -239,52 +239,38 @@ class Q4Decoder:
         check(lib().tlb_decoder_ipc_open(self.h, blob))
         dist.barrier(group=group)
 
-    # ---- running ---------------------------------------------------------------
-    def set_pos(self, pos):
-        check(lib().tlb_decoder_set_pos(self.h, pos, self._stream()))
-
-    def set_token(self, tok):
-        check(lib().tlb_decoder_set_token(self.h, int(tok), self._stream()))
-
-    def forward(self):
-        check(lib().tlb_decoder_forward(self.h, self._stream()))
-
-    def capture(self):
-        check(lib().tlb_decoder_capture(self.h))
-        self.captured = True
-
-    def run(self, n):
-        check(lib().tlb_decoder_run(self.h, n, self._stream()))
-
-    def step(self, token=None):
-        """One token end to end with host buffers: id in, next id out."""
-        tin = C.c_int32(-1 if token is None else int(token))
-        tout = C.c_int32(0)
-        check(lib().tlb_decoder_step(self.h, C.byref(tin), C.byref(tout), self._stream()))
-        return int(tout.value)
-
-    def prefill(self, tokens):
-        """prefill_batched (bench/cuda/qwen_model.h:423-442): the whole prompt as row-batched
-        GEMMs + tiled causal attention from the current position; returns the greedy next
-        token, which is also left on the device for run()."""
-        ids = (C.c_int32 * len(tokens))(*[int(t) for t in tokens])
-        tout = C.c_int32(0)
-        check(lib().tlb_decoder_prefill(self.h, ids, len(tokens), C.byref(tout), self._stream()))
-        return int(tout.value)
-
-    def last_token(self):
-        t = C.c_int32(0)
-        check(lib().tlb_decoder_last_token(self.h, C.byref(t), self._stream()))
-        return int(t.value)
-
-    def launches_per_token(self):
-        return int(lib().tlb_decoder_launches_per_token(self.h))
-
     def close(self):
-        if self.h:
-            check(lib().tlb_decoder_destroy(self.h))
-            self.h = None
-            self._keep.clear()
+        super().close()
+        self._keep.clear()
+
+    @classmethod
+    def from_folder(cls, config, tensors, dtype, max_ctx):
+        """A Qwen2-architecture checkpoint: every linear quantised to q4 on the device, norms and
+        embedding f32; `dtype` is the type of the KV caches."""
+        n_q = config["num_attention_heads"]
+        cfg = dict(hidden=config["hidden_size"], layers=config["num_hidden_layers"], n_q=n_q,
+                   n_kv=config.get("num_key_value_heads", n_q), hd=config["hidden_size"] // n_q,
+                   ff=config["intermediate_size"], vocab=config["vocab_size"], eps=config["rms_norm_eps"],
+                   rope_base=config["rope_theta"])
+        d = cls(cfg, max_ctx, kv_dtype="bf16" if dtype == "bfloat16" else "f32")
+        dev = lambda *names: torch.from_numpy(np.concatenate([tensors.f32(n) for n in names])).cuda()
+        kn = lambda *names: dev(*names).t().contiguous()
+        d.set_vector_full(0, "embed", dev("model.embed_tokens.weight"))
+        d.set_vector_full(0, "onorm", dev("model.norm.weight"))
+        tied = "lm_head.weight" not in tensors
+        d.set_linear_full(0, "lm_head", kn("model.embed_tokens.weight" if tied else "lm_head.weight"))
+        for l in range(cfg["layers"]):
+            p = f"model.layers.{l}."
+            a = p + "self_attn."
+            d.set_linear_full(l, "wqkv", kn(a + "q_proj.weight", a + "k_proj.weight", a + "v_proj.weight"))
+            d.set_linear_full(l, "wo", kn(a + "o_proj.weight"))
+            d.set_linear_full(l, "wgu", kn(p + "mlp.gate_proj.weight", p + "mlp.up_proj.weight"))
+            d.set_linear_full(l, "wd", kn(p + "mlp.down_proj.weight"))
+            d.set_vector_full(l, "an", dev(p + "input_layernorm.weight"))
+            d.set_vector_full(l, "fn", dev(p + "post_attention_layernorm.weight"))
+            for name, v in (("bq", "q_proj"), ("bk", "k_proj"), ("bv", "v_proj")):
+                d.set_vector_full(l, name, dev(a + v + ".bias"))
+        return d
 
 
 class _Ext:

@@ -261,10 +261,70 @@ int tlb_decoder_run(void* dec, int64_t n_tokens, void* stream);        /* qm:862
 /* qm:747-752 step_imperative with HOST buffers: token id in, next id out. */
 int tlb_decoder_step(void* dec, const int32_t* token_in, int32_t* token_out, void* stream);
 int tlb_decoder_last_token(void* dec, int32_t* token_out, void* stream);
-/* qm:357-442 prefill_chunk_ / prefill_batched: T prompt tokens (HOST ids) as row-batched GEMMs on
- * the int4 weights + tiled causal attention, in chunks of 1024 (TLB_PREFILL_CHUNK overrides), from the current position; leaves
- * position += T and the greedy next token on the device and in *next_token.  Single GPU. */
+/* qm:357-442 prefill_chunk_ / prefill_batched: T prompt tokens (HOST ids) as row-batched GEMMs +
+ * tiled causal attention, in passes of the model's own row count (TLB_PREFILL_CHUNK overrides), from
+ * the current position; leaves position += T and the greedy next token on the device and in
+ * *next_token.  Single GPU. */
 int tlb_decoder_prefill(void* dec, const int32_t* tokens, int64_t T, int32_t* next_token, void* stream);
+/* The same pass, which also returns the logits at `n_want` places of it: `want` is increasing, in
+ * [0, T); logits_out is HOST memory [n_want, vocab].  No counterpart in the reference (its prefill
+ * keeps the last row only). */
+int tlb_decoder_prefill_logits(void* dec, const int32_t* tokens, int64_t T, const int32_t* want, int64_t n_want,
+                               float* logits_out, int32_t* next_token, void* stream);
+
+/* ---- layer-stack decoder: a list of layers, each with one or two sequence mixers over the same
+ * normed input and an optional feed-forward, on the tlb_decoder_* sequence surface above (set_pos,
+ * set_token, forward, capture, run, step, prefill, prefill_logits, last_token, logits, destroy).
+ * No counterpart in the reference.  Weights are bf16 (f32 = 0) or f32 (f32 = 1), everything else f32;
+ * with f32 weights every product is a true 32-bit one.
+ *
+ * Carried per sequence: keys and values of the last `window` positions and of the first `keep_first`
+ * ones, a recurrent state [heads][dim][vdim] in f32, the last `conv` inputs of each convolution.  All
+ * of it is addressed by position, so tlb_decoder_set_pos(dec, 0) starts a new sequence; any other
+ * move than to the current position is refused.
+ *
+ * The projected row of a layer is the mixers' parts one after the other, every part padded to a
+ * multiple of 8 rows (zero weight rows):
+ *   attention   q [heads*dim] | k [kv_heads*dim] | v [kv_heads*vdim] | gate [heads*vdim]
+ *   delta rule  q [kv_heads*dim] | k [kv_heads*dim] | v [heads*vdim] | gate [heads*vdim] | b [heads] | a [heads]
+ *   ssd         z [heads*vdim] | x,B,C [heads*vdim + 2*kv_heads*dim] (one part) | dt [heads]
+ * Convolution weights cover the padded channels of q | k | v, or of x,B,C.  The row the output
+ * projection reads is the mixers' heads, [heads*vdim] each, padded to multiples of 8. ---- */
+#define TLB_MIX_ATTN 1
+#define TLB_MIX_DELTA 2
+#define TLB_MIX_SSD 3
+typedef struct {
+  int32_t kind;
+  int32_t heads, kv_heads;        /* ssd: kv_heads = groups */
+  int32_t dim, vdim;              /* ssd: dim = state width */
+  int32_t window, keep_first;     /* attention */
+  int32_t rot_dims;
+  int32_t conv;                   /* taps, recurrent mixers */
+  int32_t norm_groups;            /* ssd */
+  float rot_base, scale;          /* attention */
+  float out_scale;                /* factor of the mixer's result in the layer */
+} tlb_mixer_cfg;
+typedef struct {
+  int32_t n_mixers;
+  int32_t ff;                     /* 0: no feed-forward */
+  float limit;                    /* clipped gated unit */
+  tlb_mixer_cfg mixer[2];
+} tlb_layer_cfg;
+typedef struct {
+  int32_t width, vocab, n_layers, max_ctx, f32;
+  float eps, embed_scale;
+} tlb_stack_cfg;
+int tlb_stack_create(const tlb_stack_cfg* cfg, const tlb_layer_cfg* layers, void** out);
+/* HOST matrices [rows, cols] in the model's type, copied to the device.  which: 0 input projection,
+ * 1 output projection, 2 gate and up rows interleaved [2*ff, width], 3 down [width, ff], 4 embedding
+ * [vocab, width] (also the output head; layer ignored). */
+int tlb_stack_set_matrix(void* dec, int64_t layer, int which, const void* w, int64_t rows, int64_t cols);
+/* HOST f32 vectors.  which: 0 norm in front of the mixers, 1 norm in front of the feed-forward,
+ * 2 final norm (layer ignored); of mixer m: 10 + query norm 0, key norm 1, output norm 2,
+ * convolution weights [channels, taps] 3, convolution bias 4, step bias 5, log decay rate 6, skip 7. */
+int tlb_stack_set_vector(void* dec, int64_t layer, int mixer, int which, const float* v, int64_t n);
+/* Bytes of sequence state (caches, rings, recurrent states) the decoder holds. */
+int64_t tlb_stack_state_bytes(void* dec);
 /* Tensor-parallel wiring (no counterpart in the reference, which is single-device):
  * each rank exports a 128-byte record, the ranks exchange them over any host
  * channel, and every rank opens the others' exchange buffers. */
