@@ -286,6 +286,91 @@ def config_block(n):
                 l2="inputs larger than L2 (4.4 GB of weights streamed per token vs 126 MB L2)")
 
 
+# ------------------------------------------------------------- other models (--model)
+def zavilorn_config(size):
+    """Layers of a real model's proportions: one 'parallel' layer with its feed-forward for every
+    three 'mamba2' layers."""
+    w, heads, kv, ff = dict(small=(2048, 16, 4, 5632), medium=(4096, 32, 8, 14336))[size]
+    par = dict(type="parallel", mlp=dict(kind="dense", ff=ff, limit=7.0), mixer=dict(
+        left=dict(heads=heads, kv_heads=kv, dim=128, vdim=128, mask=dict(size=2048, keep_first=4),
+                  rot=dict(base=1e5, dims=64), scale=128 ** -0.5),
+        right=dict(heads=heads, kv_heads=heads // 2, dim=128, vdim=128, conv=4), left_scale=1.0, right_scale=0.5))
+    mam = dict(type="mamba2", mlp=None, mixer=dict(heads=w // 32, groups=8, state=128, vdim=64, conv=4, norm_groups=8))
+    return dict(architecture="Zavilorn", vocab=65536, width=w, embedding=dict(scale=1.0), norm=dict(eps=1e-6),
+                layers=[par, mam, mam, mam] * 2)
+
+
+def run_model(args):
+    """Prefill and decode throughput of the layer-stack model (random weights, one GPU) beside the int4
+    decoder with the same width, heads, feed-forward, vocabulary and layer count.  One JSON line per size."""
+    import torch
+    from cpp_tensorlib_b200.zavilorn import RandomTensors, Zavilorn
+    torch.cuda.set_device(0)
+    T, K, W = args.prefill or 4096, args.steps, max(3, args.warmup)
+    peak, src = measured_peaks()
+    for size in args.size.split(","):
+        cfg = zavilorn_config(size)
+        a = cfg["layers"][0]["mixer"]["left"]
+        qcfg = dict(hidden=cfg["width"], layers=len(cfg["layers"]), n_q=a["heads"], n_kv=a["kv_heads"], hd=128,
+                    ff=cfg["layers"][0]["mlp"]["ff"], vocab=cfg["vocab"], eps=1e-6, rope_base=1e6)
+        ids = np_ids(cfg["vocab"], T)
+        line = dict(metric="prefill and decode tok/s", size=size, prompt=T, steps=K, warmup=W, n_gpus=1, data="synthetic",
+                    config=dict(zavilorn=cfg, q4=qcfg), peak_source=src)
+
+        def measure(d):
+            times = []
+            for _ in range(2 + max(1, args.repeats)):
+                d.set_pos(0)
+                torch.cuda.synchronize()
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                e0.record()
+                d.prefill(ids)
+                e1.record()
+                torch.cuda.synchronize()
+                times.append(e0.elapsed_time(e1))
+            pre = statistics.median(times[2:])
+            d.capture()
+            d.run(W)
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            torch.cuda.synchronize()
+            e0.record()
+            d.run(K)
+            e1.record()
+            torch.cuda.synchronize()
+            dec = e0.elapsed_time(e1) / K
+            return dict(prefill_ms=pre, prefill_tok_s=T / pre * 1e3, decode_ms=dec, decode_tok_s=1e3 / dec,
+                        launches_per_token=d.launches_per_token())
+
+        with ClockSampler(0) as clk:
+            z = Zavilorn(cfg, "bfloat16", T + W + K + 8)
+            t = RandomTensors(cfg, SEED)
+            z.load(t)
+            mats = sum(s[0] * s[1] for n, s in t.shapes.items() if len(s) == 2 and not n.endswith("conv"))
+            r = measure(z)
+            z.close()
+            win = sum(2 * a["kv_heads"] * 128 * 2 * min(T, a["mask"]["size"] + 4) for L in cfg["layers"] if L["type"] == "parallel")
+            rec = sum(2 * 4 * (m["heads"] * m["vdim"] * m["state"] if L["type"] == "mamba2" else
+                               m["right"]["heads"] * 128 * 128) for L in cfg["layers"] for m in [L["mixer"]])
+            r.update(decode_bytes=2 * mats + win + rec, decode_frac_hbm=(2 * mats + win + rec) / r["decode_ms"] / 1e6 / peak,
+                     prefill_matrix_tflops=2 * (mats - cfg["vocab"] * cfg["width"]) * T / r["prefill_ms"] / 1e9)
+            line["zavilorn"] = r
+            if not args.no_q4:
+                q = build_decoder(qcfg, T + W + K + 8, 0, 1, 0)
+                r = measure(q)
+                q.close()
+                wb, kv, params = token_bytes(qcfg, T)
+                r.update(decode_bytes=wb + kv, decode_frac_hbm=(wb + kv) / r["decode_ms"] / 1e6 / peak,
+                         prefill_matrix_tflops=2 * (params - cfg["vocab"] * cfg["width"]) * T / r["prefill_ms"] / 1e9)
+                line["q4"] = r
+        line["clocks"] = clk.summary()
+        print(json.dumps(line), flush=True)
+
+
+def np_ids(vocab, n):
+    import numpy as np
+    return [int(v) for v in np.random.default_rng(SEED).integers(0, vocab, n)]
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -296,12 +381,19 @@ def main():
     ap.add_argument("--prefill", type=int, default=0,
                     help="diagnostic: time the batched prompt pass over this many tokens and exit")
     ap.add_argument("--no-cpu-baseline", action="store_true")
+    ap.add_argument("--model", default="q4", choices=["q4", "zavilorn"],
+                    help="zavilorn: prefill and decode of the layer-stack model beside the int4 decoder, then exit")
+    ap.add_argument("--size", default="small,medium", help="with --model zavilorn: sizes, with commas between them")
+    ap.add_argument("--repeats", type=int, default=5, help="with --model zavilorn: timed prompt passes")
+    ap.add_argument("--no-q4", action="store_true", help="with --model zavilorn: leave the int4 decoder out")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local = int(os.environ.get("LOCAL_RANK", "0"))
     if args.impl == "reference":
         return run_reference(args, rank)
+    if args.model != "q4":
+        return run_model(args)
 
     import torch
     import torch.distributed as dist

@@ -33,7 +33,8 @@ struct AttnP {
   int oa;                      // part of the finished row
   long long cap, ring;         // cache rows per head = kept slots + ring
   float scale, eps, out_scale;
-  const float *qn, *kn, *inv_freq;
+  const float *qn, *kn;
+  const float2* inv_freq;      // [pairs] angular frequencies, high and low parts
   void *K, *V;                 // [G][cap][Dp], [G][cap][Ep]
   int splits, hb, hpb;         // key ranges of a token, head blocks of a group, heads per block
   float* part;                 // [G*hb][splits][hpb][E + 2]
@@ -120,6 +121,17 @@ __device__ __forceinline__ Visible visible_of(const AttnP& p, int pos) {
 }
 __device__ __forceinline__ int visible_pos(const Visible& v, int t) { return t < v.kept ? t : v.lo + (t - v.kept); }
 
+// sine and cosine of pos * f.  The rounding of an f32 product grows with the position (one part in
+// 2^24 of hundreds of radians), so its remainder is carried along and applied as a small rotation.
+__device__ __forceinline__ void rot_angle(int pos, float2 f, float* sn, float* cs) {
+  const float a = (float)pos * f.x;
+  const float r = fmaf((float)pos, f.x, -a) + (float)pos * f.y;
+  float s, c;
+  sincosf(a, &s, &c);
+  *sn = fmaf(r, c, s);
+  *cs = fmaf(-r, s, c);
+}
+
 // one element of a normed and rotated query or key head: src points at the head's raw values, w at
 // its norm weights, rinv is 1 / rms of the whole projection
 __device__ __forceinline__ float rot_elem(const AttnP& p, const float* src, const float* w, float rinv, int pos, int d) {
@@ -127,7 +139,7 @@ __device__ __forceinline__ float rot_elem(const AttnP& p, const float* src, cons
   const int e = d & ~1;
   const float u = src[e] * rinv * w[e], v = src[e + 1] * rinv * w[e + 1];
   float sn, cs;
-  sincosf((float)pos * p.inv_freq[d >> 1], &sn, &cs);
+  rot_angle(pos, p.inv_freq[d >> 1], &sn, &cs);
   return (d & 1) ? v * cs + u * sn : u * cs - v * sn;
 }
 
@@ -245,13 +257,17 @@ __device__ __forceinline__ float conv_silu(const ConvP& p, const float* cur, lon
   return silu_f(y);
 }
 
+// exp(-x) of a decay that is applied once per token: near 1 it is rounded from an exact complement,
+// so that hundreds of factors do not add up the exponential's own last-place error.
+__device__ __forceinline__ float decay_of(float x) { return x < 0.5f ? 1.0f + expm1f(-x) : expf(-x); }
+
 // step size and decay of head h: (beta, g) of the delta rule, (dt, decay) of ssd
 __device__ __forceinline__ float2 recur_gates(const RecurP& p, const float* row, int h) {
   if (p.kind == MIX_DELTA)
     return make_float2(sigmoid_f(row[p.ob + h]),
-                       expf(-expf(p.A_log[h]) * softplus_f(row[p.oa_ + h] + p.dt_bias[h])));
+                       decay_of(expf(p.A_log[h]) * softplus_f(row[p.oa_ + h] + p.dt_bias[h])));
   const float dt = softplus_f(row[p.ob + h] + p.dt_bias[h]);
-  return make_float2(dt, expf(-expf(p.A_log[h]) * dt));
+  return make_float2(dt, decay_of(expf(p.A_log[h]) * dt));
 }
 
 #endif  // __CUDACC__

@@ -287,12 +287,16 @@ static int build(StackDecoder* d, const tlb_stack_cfg* cfg, const tlb_layer_cfg*
         if (p.splits > MX_TK) p.splits = MX_TK;
         if (!rc) rc = d->alloc((void**)&p.part, (size_t)units * p.splits * p.hpb * (p.Ep + 2) * 4, d->owned);
         if (!rc) rc = d->alloc((void**)&p.counters, (size_t)units * sizeof(int), d->owned);
-        std::vector<float> f(max_i(1, p.pairs));
-        for (int i = 0; i < p.pairs; i++) f[i] = (float)pow((double)k.rot_base, -2.0 * i / k.rot_dims);
-        float* df = nullptr;
-        if (!rc) rc = d->alloc((void**)&df, f.size() * 4, d->owned);
+        std::vector<float2> f(max_i(1, p.pairs));
+        for (int i = 0; i < p.pairs; i++) {
+          const double w = pow((double)k.rot_base, -2.0 * i / k.rot_dims);
+          f[i].x = (float)w;
+          f[i].y = (float)(w - (double)f[i].x);
+        }
+        float2* df = nullptr;
+        if (!rc) rc = d->alloc((void**)&df, f.size() * sizeof(float2), d->owned);
         if (rc) return rc;
-        TLB_CUDA(cudaMemcpy(df, f.data(), f.size() * 4, cudaMemcpyHostToDevice));
+        TLB_CUDA(cudaMemcpy(df, f.data(), f.size() * sizeof(float2), cudaMemcpyHostToDevice));
         p.inv_freq = df;
         d->q_max = max_i(d->q_max, H * p.Dp);
       } else if (k.kind == TLB_MIX_DELTA || k.kind == TLB_MIX_SSD) {

@@ -6,6 +6,7 @@ mixers.  Every size and constant comes from the configuration.
 """
 import numpy as np
 
+from .safetensors import bf16_to_f32, f32_to_bf16
 from .stack import ATTN, DELTA, SSD, LayerStack, mixer_cfg, pad_rows
 
 
@@ -84,3 +85,68 @@ class Zavilorn(LayerStack):
         self.set_vector(i, "conv_bias", pad_rows(t.f32(p + "conv.b")))
         for name, key in (("dt_bias", "dt_bias"), ("A_log", "A_log"), ("skip", "D"), ("norm", "norm")):
             self.set_vector(i, name, t.f32(p + key))
+
+
+def tensor_shapes(config):
+    """name -> shape of every tensor of a model with this configuration."""
+    w, out = config["width"], {"embed": (config["vocab"], config["width"]), "final.norm": (config["width"],)}
+    for i, entry in enumerate(config["layers"]):
+        p, m = f"l{i}.", entry["mixer"]
+        out[p + "norm1"] = (w,)
+        if entry["type"] == "parallel":
+            a, d, l, r = m["left"], m["right"], p + "mix.left.", p + "mix.right."
+            q, k = a["heads"] * a["dim"], a["kv_heads"] * a["dim"]
+            v, o = a["kv_heads"] * a["vdim"], a["heads"] * a["vdim"]
+            out.update({l + "q": (q, w), l + "k": (k, w), l + "v": (v, w), l + "g": (o, w), l + "o": (w, o),
+                        l + "q.norm": (q,), l + "k.norm": (k,)})
+            q, o, h = d["kv_heads"] * d["dim"], d["heads"] * d["vdim"], d["heads"]
+            for n, rows in (("q", q), ("k", q), ("v", o)):
+                out.update({r + n: (rows, w), r + n + ".conv": (rows, d["conv"])})
+            out.update({r + "b": (h, w), r + "a": (h, w), r + "A_log": (h,), r + "dt_bias": (h,),
+                        r + "norm": (d["vdim"],), r + "g": (o, w), r + "o": (w, o)})
+        else:
+            h, inner = m["heads"], m["heads"] * m["vdim"]
+            c = inner + 2 * m["groups"] * m["state"]
+            p2 = p + "mix."
+            out.update({p2 + "in": (inner + c + h, w), p2 + "conv": (c, m["conv"]), p2 + "conv.b": (c,),
+                        p2 + "dt_bias": (h,), p2 + "A_log": (h,), p2 + "D": (h,), p2 + "norm": (inner,),
+                        p2 + "o": (w, inner)})
+        if entry.get("mlp"):
+            f = entry["mlp"]["ff"]
+            out.update({p + "norm2": (w,), p + "mlp.gate": (f, w), p + "mlp.up": (f, w), p + "mlp.down": (w, f)})
+    return out
+
+
+class RandomTensors:
+    """Random weights of a configuration, slices of one pool of normal numbers (raw() and f32() of a
+    SafeTensors).  Matrices have standard deviation 1 / sqrt(columns), norms are near one, decay rates
+    and step biases lie where the recurrences remember tens to hundreds of tokens."""
+
+    def __init__(self, config, seed=0, pool=1 << 24):
+        self.shapes = tensor_shapes(config)
+        self.rng = np.random.default_rng(seed)
+        self.pool = self.rng.standard_normal(pool, dtype=np.float32)
+
+    def __contains__(self, name):
+        return name in self.shapes
+
+    def names(self):
+        return list(self.shapes)
+
+    def f32(self, name):
+        shape = self.shapes[name]
+        n = int(np.prod(shape))
+        at = int(self.rng.integers(len(self.pool)))
+        a = np.resize(np.roll(self.pool, -at) if n > len(self.pool) - at else self.pool[at:at + n], shape)
+        if name.endswith("norm") or name.endswith(("norm1", "norm2")):
+            a = 1.0 + 0.1 * a
+        elif name.endswith("A_log"):
+            a = 0.3 * a
+        elif name.endswith("dt_bias"):
+            a = -3.0 + 0.5 * a
+        elif len(shape) == 2 and name != "embed":
+            a = a / np.float32(np.sqrt(shape[1]))
+        return bf16_to_f32(f32_to_bf16(a)).reshape(shape)
+
+    def raw(self, name):
+        return f32_to_bf16(self.f32(name))
