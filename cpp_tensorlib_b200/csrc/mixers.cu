@@ -28,7 +28,70 @@ struct DecodeArgs {
 };
 
 // ---- attention, one token ------------------------------------------------------------------
+// Everything but the projected row was written at least two launches ago, and the launch before this
+// one starts its successors only behind its own wait: the position, the caches, the states and the
+// weights may be read before pdl_wait.
+struct AttnUnit {
+  int g, gb, h0, nh, split, active, t0, t1;
+  Visible vis;
+};
+__device__ __forceinline__ AttnUnit attn_unit_of(const AttnP& p, int unit, int pos) {
+  AttnUnit a;
+  a.split = unit % p.splits;
+  a.gb = unit / p.splits;
+  a.g = a.gb / p.hb;
+  a.h0 = a.g * (p.H / p.G) + (a.gb % p.hb) * p.hpb;
+  const int left = (a.g + 1) * (p.H / p.G) - a.h0;
+  a.nh = left < p.hpb ? left : p.hpb;
+  a.vis = visible_of(p, pos);
+  int chunk = (a.vis.n + p.splits - 1) / p.splits;
+  chunk = chunk < 64 ? 64 : chunk;
+  a.active = (a.vis.n + chunk - 1) / chunk;
+  a.t0 = a.split * chunk;
+  a.t1 = a.t0 + chunk < a.vis.n ? a.t0 + chunk : a.vis.n;
+  return a;
+}
+// normed and rotated query heads of the unit into qs [RM][Dp]; with the range that ends with the token
+// itself, its key and value into the cache and (bf16 values) into knew [Dp] | [Ep]
 template <typename KT, int RM>
+__device__ void attn_token_heads(const AttnP& p, const AttnUnit& a, const float* row, int pos, const float2* cs,
+                                 float* qs, KT* knew, float* red) {
+  const int tid = threadIdx.x;
+  const bool last = a.split == a.active - 1;
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < p.H * p.D; i += MX_THREADS) { const float v = row[p.oq + i]; sq = fmaf(v, v, sq); }
+  if (last)
+    for (int i = tid; i < p.G * p.D; i += MX_THREADS) { const float v = row[p.ok + i]; sk = fmaf(v, v, sk); }
+  sq = block_sum(sq, red);
+  const float rq = rsqrtf(sq / (p.H * p.D) + p.eps);
+  for (int i = tid; i < RM * p.Dp; i += MX_THREADS) {
+    const int r = i / p.Dp, d = i - r * p.Dp;
+    float v = 0.f;
+    if (r < a.nh && d < p.D) v = rot_elem(p, row + p.oq + (a.h0 + r) * p.D, p.qn + (a.h0 + r) * p.D, rq, cs, d);
+    if (sizeof(KT) == 2) v = __bfloat162float(__float2bfloat16_rn(v));
+    qs[i] = v;
+  }
+  if (last) {
+    sk = block_sum(sk, red);
+    const float rk = rsqrtf(sk / (p.G * p.D) + p.eps);
+    const size_t slot = kv_slot(p, pos);
+    KT* kd = (KT*)p.K + ((size_t)a.g * p.cap + slot) * p.Dp;
+    KT* vd = (KT*)p.V + ((size_t)a.g * p.cap + slot) * p.Ep;
+    for (int d = tid; d < p.Dp; d += MX_THREADS) {
+      const float v = d < p.D ? rot_elem(p, row + p.ok + a.g * p.D, p.kn + a.g * p.D, rk, cs, d) : 0.f;
+      put(kd + d, v);
+      put(knew + d, v);
+    }
+    for (int e = tid; e < p.Ep; e += MX_THREADS) {
+      const float v = e < p.E ? row[p.ov + a.g * p.E + e] : 0.f;
+      put(vd + e, v);
+      put(knew + p.Dp + e, v);
+    }
+  }
+  __syncthreads();
+}
+
+template <int RM>
 __device__ void attn_finish(const AttnP& p, const float* os, const float* ml, int h0, int nh, const float* row,
                             float* out) {
   for (int i = threadIdx.x; i < nh * p.E; i += MX_THREADS) {
@@ -36,69 +99,32 @@ __device__ void attn_finish(const AttnP& p, const float* os, const float* ml, in
     out[p.oa + c] = os[r * p.Ep + e] / ml[RM + r] * sigmoid_f(row[p.og + c]) * p.out_scale;
   }
 }
-
-template <typename KT, int RM>
-__device__ void attn_decode_unit(const AttnP& p, int unit, const float* row, float* out, int pos, float* sm) {
+// a range's unnormalised heads (os), maxima and sums (ml) into the partials; the last range to arrive
+// merges them all
+template <int RM>
+__device__ void attn_merge(const AttnP& p, const AttnUnit& a, float* os, float* ml, float* sc, const float* row,
+                           float* out) {
   __shared__ int s_last;
-  float* qs = sm;                         // [RM][Dp]
-  float* os = qs + RM * p.Dp;             // [RM][Ep]
-  float* sc = os + RM * p.Ep;             // [RM][MX_TK]
-  float* ml = sc + RM * MX_TK;            // [3][RM]
-  float* red = ml + 3 * RM;               // [33]
-  const int tid = threadIdx.x, split = unit % p.splits, gb = unit / p.splits;
-  const int g = gb / p.hb, h0 = g * (p.H / p.G) + (gb % p.hb) * p.hpb;
-  const int left = (g + 1) * (p.H / p.G) - h0, nh = left < p.hpb ? left : p.hpb;
-  const Visible vis = visible_of(p, pos);
-  int chunk = (vis.n + p.splits - 1) / p.splits;
-  chunk = chunk < 64 ? 64 : chunk;
-  const int active = (vis.n + chunk - 1) / chunk;
-  if (split >= active) return;
-  const int t0 = split * chunk, t1 = t0 + chunk < vis.n ? t0 + chunk : vis.n;
-
-  float sq = 0.f;
-  for (int i = tid; i < p.H * p.D; i += MX_THREADS) { const float v = row[p.oq + i]; sq = fmaf(v, v, sq); }
-  sq = block_sum(sq, red);
-  const float rq = rsqrtf(sq / (p.H * p.D) + p.eps);
-  for (int i = tid; i < RM * p.Dp; i += MX_THREADS) {
-    const int r = i / p.Dp, d = i - r * p.Dp;
-    float v = 0.f;
-    if (r < nh && d < p.D) v = rot_elem(p, row + p.oq + (h0 + r) * p.D, p.qn + (h0 + r) * p.D, rq, pos, d);
-    if (sizeof(KT) == 2) v = __bfloat162float(__float2bfloat16_rn(v));
-    qs[i] = v;
-  }
-  if (split == active - 1) {   // this range ends with the token itself: put its key and value down first
-    float sk = 0.f;
-    for (int i = tid; i < p.G * p.D; i += MX_THREADS) { const float v = row[p.ok + i]; sk = fmaf(v, v, sk); }
-    sk = block_sum(sk, red);
-    const float rk = rsqrtf(sk / (p.G * p.D) + p.eps);
-    const long long slot = kv_slot(p, pos);
-    KT* kd = (KT*)p.K + ((size_t)g * p.cap + slot) * p.Dp;
-    KT* vd = (KT*)p.V + ((size_t)g * p.cap + slot) * p.Ep;
-    for (int d = tid; d < p.D; d += MX_THREADS)
-      put(kd + d, rot_elem(p, row + p.ok + g * p.D, p.kn + g * p.D, rk, pos, d));
-    for (int e = tid; e < p.E; e += MX_THREADS) put(vd + e, row[p.ov + g * p.E + e]);
-  }
-  __syncthreads();
-  attn_range<KT, RM>(p, qs, g, vis, t0, t1, sc, os, ml);
+  const int tid = threadIdx.x, nh = a.nh, active = a.active;
   if (active == 1) {
-    attn_finish<KT, RM>(p, os, ml, h0, nh, row, out);
+    attn_finish<RM>(p, os, ml, a.h0, nh, row, out);
     return;
   }
   const int PS = p.Ep + 2;
-  float* part = p.part + (size_t)gb * p.splits * p.hpb * PS;
+  float* part = p.part + (size_t)a.gb * p.splits * p.hpb * PS;
   for (int i = tid; i < nh * p.Ep; i += MX_THREADS)
-    part[((size_t)split * p.hpb + i / p.Ep) * PS + i % p.Ep] = os[i];
+    part[((size_t)a.split * p.hpb + i / p.Ep) * PS + i % p.Ep] = os[i];
   if (tid < nh) {
-    part[((size_t)split * p.hpb + tid) * PS + p.Ep] = ml[tid];
-    part[((size_t)split * p.hpb + tid) * PS + p.Ep + 1] = ml[RM + tid];
+    part[((size_t)a.split * p.hpb + tid) * PS + p.Ep] = ml[tid];
+    part[((size_t)a.split * p.hpb + tid) * PS + p.Ep + 1] = ml[RM + tid];
   }
   __threadfence();
   __syncthreads();
-  if (tid == 0) s_last = atomicAdd(&p.counters[gb], 1) == active - 1;
+  if (tid == 0) s_last = atomicAdd(&p.counters[a.gb], 1) == active - 1;
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  if (tid == 0) p.counters[gb] = 0;
+  if (tid == 0) p.counters[a.gb] = 0;
   const int warp = tid >> 5, lane = tid & 31;
   for (int r = warp; r < nh; r += MX_THREADS / 32) {
     float m = -3.0e38f;
@@ -116,31 +142,264 @@ __device__ void attn_decode_unit(const AttnP& p, int unit, const float* row, flo
   __syncthreads();
   for (int i = tid; i < nh * p.Ep; i += MX_THREADS) {
     const int r = i / p.Ep, e = i - r * p.Ep;
-    float a = 0.f;
-    for (int s = 0; s < active; s++) a = fmaf(sc[r * MX_TK + s], __ldcg(&part[((size_t)s * p.hpb + r) * PS + e]), a);
-    os[i] = a;
+    const float* src = part + (size_t)r * PS + e;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    int s = 0;
+    for (; s + 8 <= active; s += 8) {
+      float v[8];
+#pragma unroll
+      for (int k = 0; k < 8; k++) v[k] = __ldcg(src + (size_t)(s + k) * p.hpb * PS);
+#pragma unroll
+      for (int k = 0; k < 8; k++) acc[k & 3] = fmaf(sc[r * MX_TK + s + k], v[k], acc[k & 3]);
+    }
+    for (; s < active; s++) acc[0] = fmaf(sc[r * MX_TK + s], __ldcg(src + (size_t)s * p.hpb * PS), acc[0]);
+    os[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
   }
   __syncthreads();
-  attn_finish<KT, RM>(p, os, ml, h0, nh, row, out);
+  attn_finish<RM>(p, os, ml, a.h0, nh, row, out);
+}
+
+// any widths, either cache type
+template <typename KT, int RM>
+__device__ void attn_decode_unit(const AttnP& p, int unit, const float* row, float* out, int pos, float* sm) {
+  __shared__ float2 cs[MX_PAIRS];
+  float* qs = sm;                         // [RM][Dp]
+  float* os = qs + RM * p.Dp;             // [RM][Ep]
+  float* sc = os + RM * p.Ep;             // [RM][MX_TK]
+  float* ml = sc + RM * MX_TK;            // [3][RM], 32
+  float* red = ml + 32;                   // [33], 40
+  KT* knew = (KT*)(red + 40);             // [Dp + Ep]
+  const AttnUnit a = attn_unit_of(p, unit, pos);
+  if (a.split >= a.active) { pdl_wait(); return; }
+  rot_table(p, pos, cs);
+  pdl_wait();
+  pdl_launch_dependents();
+  __syncthreads();
+  attn_token_heads<KT, RM>(p, a, row, pos, cs, qs, knew, red);
+  attn_range<KT, RM>(p, qs, a.g, a.vis, a.t0, a.t1, sc, os, ml);
+  attn_merge<RM>(p, a, os, ml, sc, row, out);
+}
+
+// v[N] per lane, summed over the 16 lanes of a half warp: N >= 16 leaves N / 16 sums in each lane (sum i in
+// lane i % 16 of v[i / 16]), fewer leave each sum in several lanes.  Returns the index base of the lane.
+template <int N>
+__device__ __forceinline__ int half_warp_sums(float (&v)[N]) {
+  const int lane = threadIdx.x & 31;
+  int n = N, at = 0;
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool up = lane & o;
+#pragma unroll
+      for (int i = 0; i < N / 2; i++)
+        if (i < n) {
+          const float send = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+      if (up) at += n;
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+  return at;
+}
+
+// bf16 cache, widths up to 128: 64 keys a tile, 16 lanes a key row, the first tile's keys and values in
+// flight before the projected row is there, and the next tile's under the current one's arithmetic
+constexpr int AF_TK = 64;
+template <int RM>
+__device__ void attn_decode_unit16(const AttnP& p, int unit, const float* row, float* out, int pos, float* sm) {
+  using KT = __nv_bfloat16;
+  __shared__ float2 cs[64];
+  float* qs = sm;                         // [RM][Dp]
+  float* os = qs + RM * p.Dp;             // [RM][Ep]
+  float* sc = os + RM * p.Ep;             // [RM][MX_TK]
+  float* ml = sc + RM * MX_TK;            // [3][RM], 32
+  float* red = ml + 32;                   // [33], 40
+  KT* knew = (KT*)(red + 40);             // [Dp + Ep]
+  float* wo = (float*)(knew + 256);       // [8 warps][RM][Ep]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, ch = tid & 15, kr = tid >> 4;
+  const AttnUnit a = attn_unit_of(p, unit, pos);
+  if (a.split >= a.active) { pdl_wait(); return; }
+  const KT* K = (const KT*)p.K + (size_t)a.g * p.cap * p.Dp + ch * 8;
+  const KT* V = (const KT*)p.V + (size_t)a.g * p.cap * p.Ep + ch * 8;
+  const bool ck = ch * 8 < p.Dp, cv = ch * 8 < p.Ep;
+  uint4 kf[4], vf[4];
+  auto load = [&](uint4 (&f)[4], const KT* base, int width, bool on, int tb) {
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      const int t = tb + kr + 16 * i;
+      f[i] = make_uint4(0, 0, 0, 0);
+      if (on && t < a.t1) f[i] = *(const uint4*)(base + (size_t)kv_slot(p, visible_pos(a.vis, t)) * width);
+    }
+  };
+  load(kf, K, p.Dp, ck, a.t0);
+  load(vf, V, p.Ep, cv, a.t0);
+  rot_table(p, pos, cs);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (tid < RM) { ml[tid] = -3.0e38f; ml[RM + tid] = 0.f; }
+  __syncthreads();
+  attn_token_heads<KT, RM>(p, a, row, pos, cs, qs, knew, red);
+  float acc[RM][8];
+#pragma unroll
+  for (int r = 0; r < RM; r++)
+#pragma unroll
+    for (int e = 0; e < 8; e++) acc[r][e] = 0.f;
+  for (int tb = a.t0; tb < a.t1; tb += AF_TK) {
+    const int n = a.t1 - tb < AF_TK ? a.t1 - tb : AF_TK, own = a.vis.n - 1 - tb;   // place of the token itself
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+      if (kr + 16 * i == own) {
+        if (ck) kf[i] = *(const uint4*)(knew + ch * 8);
+        if (cv) vf[i] = *(const uint4*)(knew + p.Dp + ch * 8);
+      }
+    float s[4 * RM];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      float f[8];
+      widen16(kf[i], f, (const KT*)nullptr);
+#pragma unroll
+      for (int r = 0; r < RM; r++) {
+        float d = 0.f;
+        if (ck) {
+          const float4 x = *(const float4*)(qs + r * p.Dp + ch * 8), y = *(const float4*)(qs + r * p.Dp + ch * 8 + 4);
+          d = fmaf(f[0], x.x, fmaf(f[1], x.y, fmaf(f[2], x.z, f[3] * x.w)));
+          d = fmaf(f[4], y.x, fmaf(f[5], y.y, fmaf(f[6], y.z, fmaf(f[7], y.w, d))));
+        }
+        s[i * RM + r] = d;
+      }
+    }
+    if (tb + AF_TK < a.t1) load(kf, K, p.Dp, ck, tb + AF_TK);
+    const int at = half_warp_sums<4 * RM>(s);
+    constexpr int NS = 4 * RM > 16 ? 4 * RM / 16 : 1;
+#pragma unroll
+    for (int j = 0; j < NS; j++) {
+      const int x = at + j, i = x / RM, r = x - i * RM;
+      sc[r * AF_TK + kr + 16 * i] = kr + 16 * i < n ? s[j] * p.scale : -INFINITY;
+    }
+    __syncthreads();
+    for (int r = warp; r < RM; r += MX_THREADS / 32) {
+      const float x0 = sc[r * AF_TK + lane], x1 = sc[r * AF_TK + lane + 32], old = ml[r];
+      const float m = warp_max(fmaxf(old, fmaxf(x0, x1)));
+      const float e0 = expf(x0 - m), e1 = expf(x1 - m);
+      sc[r * AF_TK + lane] = e0;
+      sc[r * AF_TK + lane + 32] = e1;
+      const float l = warp_sum(e0 + e1);
+      if (lane == 0) {
+        const float c = expf(old - m);
+        ml[2 * RM + r] = c; ml[r] = m; ml[RM + r] = ml[RM + r] * c + l;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < RM; r++) {
+      const float c = ml[2 * RM + r];
+#pragma unroll
+      for (int e = 0; e < 8; e++) acc[r][e] *= c;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+      float f[8];
+      widen16(vf[i], f, (const KT*)nullptr);
+#pragma unroll
+      for (int r = 0; r < RM; r++) {
+        const float w = sc[r * AF_TK + kr + 16 * i];
+#pragma unroll
+        for (int e = 0; e < 8; e++) acc[r][e] = fmaf(w, f[e], acc[r][e]);
+      }
+    }
+    if (tb + AF_TK < a.t1) {
+      load(vf, V, p.Ep, cv, tb + AF_TK);
+      __syncthreads();   // the weights are read: the next tile's scores may overwrite them
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < RM; r++)
+#pragma unroll
+    for (int e = 0; e < 8; e++) acc[r][e] += __shfl_xor_sync(0xffffffffu, acc[r][e], 16);
+  if (lane < 16 && cv)
+#pragma unroll
+    for (int r = 0; r < RM; r++) {
+      float* d = wo + (warp * RM + r) * p.Ep + ch * 8;
+      *(float4*)d = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+      *(float4*)(d + 4) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
+    }
+  __syncthreads();
+  for (int i = tid; i < RM * p.Ep; i += MX_THREADS) {
+    float x = 0.f;
+#pragma unroll
+    for (int w = 0; w < MX_THREADS / 32; w++) x += wo[w * RM * p.Ep + i];
+    os[i] = x;
+  }
+  __syncthreads();
+  attn_merge<RM>(p, a, os, ml, sc, row, out);
 }
 
 // ---- recurrent mixers, one token -----------------------------------------------------------
+// One block a head.  A thread holds up to MX_ROWS rows of one state column, for two column blocks at a
+// time; the first two blocks and the convolutions' history are fetched before the projected row is there.
 __device__ void recur_decode_head(const RecurP& p, int h, const float* row, float* out, int pos, float* sm) {
-  const int tid = threadIdx.x, D = p.D, E = p.E, rep = p.H / p.G, kg = h / rep;
+  const int tid = threadIdx.x, D = p.D, E = p.E, rep = p.H / p.G, kg = h / rep, n = 2 * D + E;
   float* q = sm;               // [D]
   float* k = q + D;            // [D]
   float* v = k + D;            // [E]
   float* o = v + E;            // [E]
-  float* red = o + E;          // [MX_THREADS]
-  float* rs = red + MX_THREADS;  // [33]
-  const float* cur = row + p.cv.off;
-  for (int i = tid; i < 2 * D + E; i += MX_THREADS) {
-    const int c = i < D ? p.cq + kg * D + i : (i < 2 * D ? p.ck + kg * D + i - D : p.cvv + h * E + i - 2 * D);
-    sm[i] = conv_silu(p.cv, cur, 0, 0, pos, c);
-    if (p.cv.taps > 1 && (i >= 2 * D || h == kg * rep)) p.cv.ring[(size_t)(pos % p.cv.taps) * p.cv.C + c] = cur[c];
+  float* wl = o + E;           // [n] weights of the current token
+  float* red = wl + n;         // [2][MX_THREADS]
+  float* rs = red + 2 * MX_THREADS;  // [33]
+  float* S = p.S + (size_t)h * D * E;
+  const int need = (D + MX_ROWS - 1) / MX_ROWS;
+  const int VB = E < MX_THREADS / need ? E : MX_THREADS / need;
+  const int RS = MX_THREADS / VB;
+  const int grp = tid / VB, col = tid - grp * VB;
+  const size_t stride = (size_t)RS * E;
+  float s[2][MX_ROWS];
+  auto fetch = [&](int c0) {
+#pragma unroll
+    for (int b = 0; b < 2; b++) {
+      const int e = c0 + b * VB + col;
+      const int left = grp < RS && e < E && pos > 0 ? D - grp : 0;   // rows grp, grp + RS, ... below D
+      const float* at = S + (size_t)grp * E + e;
+#pragma unroll
+      for (int i = 0; i < MX_ROWS; i++) {
+        s[b][i] = i * RS < left ? *at : 0.f;
+        at += stride;
+      }
+    }
+  };
+  fetch(0);
+  auto channel = [&](int i) {
+    return i < D ? p.cq + kg * D + i : (i < 2 * D ? p.ck + kg * D + i - D : p.cvv + h * E + i - 2 * D);
+  };
+  const int taps = p.cv.taps;
+  for (int i = tid; i < n; i += MX_THREADS) {
+    const int c = channel(i);
+    const float* w = p.cv.w + (size_t)c * taps;
+    float y = p.cv.b ? p.cv.b[c] : 0.f;
+    for (int a = 0; a + 1 < taps; a++) {
+      const int qp = pos - (taps - 1 - a);
+      if (qp >= 0) y = fmaf(w[a], p.cv.ring[(size_t)(qp % taps) * p.cv.C + c], y);
+    }
+    sm[i] = y;
+    wl[i] = w[taps - 1];
   }
+  const float rate = expf(p.A_log[h]), bias = p.dt_bias[h];
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* cur = row + p.cv.off;
+  for (int i = tid; i < n; i += MX_THREADS) {
+    const int c = channel(i);
+    const float x = cur[c];
+    sm[i] = silu_f(fmaf(wl[i], x, sm[i]));
+    if (taps > 1 && (i >= 2 * D || h == kg * rep)) p.cv.ring[(size_t)(pos % taps) * p.cv.C + c] = x;
+  }
+  const bool delta = p.kind == MIX_DELTA;
+  const float step = softplus_f(row[p.oa_ + h] + bias);
+  const float in = delta ? sigmoid_f(row[p.ob + h]) : step, g = decay_of(rate * step);
   __syncthreads();
-  if (p.kind == MIX_DELTA) {
+  if (delta) {
     float sq = 0.f, sk = 0.f;
     for (int i = tid; i < D; i += MX_THREADS) { sq = fmaf(q[i], q[i], sq); sk = fmaf(k[i], k[i], sk); }
     sq = block_sum(sq, rs);
@@ -149,61 +408,78 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
     for (int i = tid; i < D; i += MX_THREADS) { q[i] *= fq; k[i] *= fk; }
     __syncthreads();
   }
-  const float2 gt = recur_gates(p, row, h);
-  float* S = p.S + (size_t)h * D * E;
-  const int need = (D + MX_ROWS - 1) / MX_ROWS;
-  const int VB = E < MX_THREADS / need ? E : MX_THREADS / need;
-  const int RS = MX_THREADS / VB;
-  const int grp = tid / VB, col = tid - grp * VB;
-  for (int c0 = 0; c0 < E; c0 += VB) {
-    const int e = c0 + col;
-    const bool on = grp < RS && e < E;
-    float s[MX_ROWS];
-    float dot = 0.f;
-#pragma unroll
-    for (int i = 0; i < MX_ROWS; i++) {
-      const int r = grp + i * RS;
-      s[i] = on && r < D && pos > 0 ? S[(size_t)r * E + e] : 0.f;
-    }
-    float u;
-    if (p.kind == MIX_DELTA) {
+  for (int c0 = 0; c0 < E; c0 += 2 * VB) {
+    if (c0) fetch(c0);
+    float u[2], acc[2] = {0.f, 0.f};
+    if (delta) {
+      float dot[2] = {0.f, 0.f};
 #pragma unroll
       for (int i = 0; i < MX_ROWS; i++) {
         const int r = grp + i * RS;
-        s[i] *= gt.y;
-        if (r < D) dot = fmaf(k[r], s[i], dot);
+        const float kk = r < D ? k[r] : 0.f;
+#pragma unroll
+        for (int b = 0; b < 2; b++) {
+          s[b][i] *= g;
+          dot[b] = fmaf(kk, s[b][i], dot[b]);
+        }
       }
-      red[tid] = dot;
+      red[tid] = dot[0];
+      red[MX_THREADS + tid] = dot[1];
       __syncthreads();
-      dot = 0.f;
-      if (on) for (int w = 0; w < RS; w++) dot += red[w * VB + col];
-      u = on ? gt.x * (v[e] - dot) : 0.f;
+#pragma unroll
+      for (int b = 0; b < 2; b++) {
+        const int e = c0 + b * VB + col;
+        float d = 0.f;
+        for (int w = 0; w < RS; w++) d += red[b * MX_THREADS + w * VB + col];
+        u[b] = grp < RS && e < E ? in * (v[e] - d) : 0.f;
+      }
       __syncthreads();
     } else {
-      u = on ? gt.x * v[e] : 0.f;
 #pragma unroll
-      for (int i = 0; i < MX_ROWS; i++) s[i] *= gt.y;
+      for (int b = 0; b < 2; b++) {
+        const int e = c0 + b * VB + col;
+        u[b] = grp < RS && e < E ? in * v[e] : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < MX_ROWS; i++) { s[0][i] *= g; s[1][i] *= g; }
     }
-    float acc = 0.f;
 #pragma unroll
     for (int i = 0; i < MX_ROWS; i++) {
       const int r = grp + i * RS;
-      if (on && r < D) {
-        s[i] = fmaf(k[r], u, s[i]);
-        acc = fmaf(q[r], s[i], acc);
-        S[(size_t)r * E + e] = s[i];
+      if (r < D) {
+        const float kk = k[r], qq = q[r];
+#pragma unroll
+        for (int b = 0; b < 2; b++) {
+          s[b][i] = fmaf(kk, u[b], s[b][i]);
+          acc[b] = fmaf(qq, s[b][i], acc[b]);
+        }
       }
     }
-    red[tid] = acc;
+    red[tid] = acc[0];
+    red[MX_THREADS + tid] = acc[1];
+#pragma unroll
+    for (int b = 0; b < 2; b++) {
+      const int e = c0 + b * VB + col;
+      const int left = grp < RS && e < E ? D - grp : 0;
+      float* at = S + (size_t)grp * E + e;
+#pragma unroll
+      for (int i = 0; i < MX_ROWS; i++) {
+        if (i * RS < left) *at = s[b][i];
+        at += stride;
+      }
+    }
     __syncthreads();
-    if (on && grp == 0) {
-      acc = 0.f;
-      for (int w = 0; w < RS; w++) acc += red[w * VB + col];
-      o[e] = acc;
+    for (int i = tid; i < 2 * VB; i += MX_THREADS) {
+      const int b = i / VB, c = i - b * VB, e = c0 + i;
+      if (e < E) {
+        float a = 0.f;
+        for (int w = 0; w < RS; w++) a += red[b * MX_THREADS + w * VB + c];
+        o[e] = a;
+      }
     }
     __syncthreads();
   }
-  if (p.kind == MIX_DELTA) {
+  if (delta) {
     float sq = 0.f;
     for (int e = tid; e < E; e += MX_THREADS) sq = fmaf(o[e], o[e], sq);
     sq = block_sum(sq, rs);
@@ -215,22 +491,21 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
   }
 }
 
-template <typename KT, int RM>
-__global__ void __launch_bounds__(MX_THREADS) mixers_decode_kernel(const __grid_constant__ DecodeArgs a) {
+template <typename KT, int RM, bool FAST>
+__global__ void __launch_bounds__(MX_THREADS, 2) mixers_decode_kernel(const __grid_constant__ DecodeArgs a) {
   extern __shared__ __align__(16) float sm[];
-  pdl_wait();
-  pdl_launch_dependents();
   const int pos = (int)*a.d_pos;
   int b = blockIdx.x;
   // recurrent heads first: they move the most bytes per block
   for (int i = 0; i < a.n_rec; i++) {
     if (b < a.rec[i].H) {
       recur_decode_head(a.rec[i], b, a.proj, a.out, pos, sm);
-      return;
+          return;
     }
     b -= a.rec[i].H;
   }
-  attn_decode_unit<KT, RM>(a.at, b, a.proj, a.out, pos, sm);
+  if (FAST) attn_decode_unit16<RM>(a.at, b, a.proj, a.out, pos, sm);
+  else attn_decode_unit<KT, RM>(a.at, b, a.proj, a.out, pos, sm);
 }
 
 // ---- prompt pass: attention ----------------------------------------------------------------
@@ -239,10 +514,12 @@ __global__ void __launch_bounds__(MX_THREADS) attn_rows_prep_kernel(const __grid
                                                                     const float* __restrict__ proj, long long ld,
                                                                     int pos0, KT* __restrict__ q) {
   __shared__ float red[33];
+  __shared__ float2 cs[MX_PAIRS];
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, tid = threadIdx.x, pos = pos0 + t;
   const float* row = proj + (size_t)t * ld;
+  rot_table(p, pos, cs);
   float sq = 0.f, sk = 0.f;
   for (int i = tid; i < p.H * p.D; i += MX_THREADS) { const float v = row[p.oq + i]; sq = fmaf(v, v, sq); }
   for (int i = tid; i < p.G * p.D; i += MX_THREADS) { const float v = row[p.ok + i]; sk = fmaf(v, v, sk); }
@@ -252,13 +529,13 @@ __global__ void __launch_bounds__(MX_THREADS) attn_rows_prep_kernel(const __grid
   KT* qd = q + (size_t)t * p.H * p.Dp;
   for (int i = tid; i < p.H * p.Dp; i += MX_THREADS) {
     const int h = i / p.Dp, d = i - h * p.Dp;
-    put(qd + i, d < p.D ? rot_elem(p, row + p.oq + h * p.D, p.qn + h * p.D, rq, pos, d) : 0.f);
+    put(qd + i, d < p.D ? rot_elem(p, row + p.oq + h * p.D, p.qn + h * p.D, rq, cs, d) : 0.f);
   }
-  const long long slot = kv_slot(p, pos);
+  const size_t slot = kv_slot(p, pos);
   for (int i = tid; i < p.G * p.D; i += MX_THREADS) {
     const int g = i / p.D, d = i - g * p.D;
     put((KT*)p.K + ((size_t)g * p.cap + slot) * p.Dp + d,
-        rot_elem(p, row + p.ok + g * p.D, p.kn + g * p.D, rk, pos, d));
+        rot_elem(p, row + p.ok + g * p.D, p.kn + g * p.D, rk, cs, d));
   }
   for (int i = tid; i < p.G * p.E; i += MX_THREADS) {
     const int g = i / p.E, e = i - g * p.E;
@@ -323,6 +600,70 @@ __global__ void __launch_bounds__(256) recur_conv_kernel(const __grid_constant__
   for (int h = threadIdx.x; h < p.H; h += blockDim.x) gates[(size_t)t * p.H + h] = recur_gates(p, row, h);
 }
 
+// The same for the chunked form: a thread runs down CT rows of two adjacent channels with the last
+// inputs in registers.
+constexpr int CV_ROWS = 32, CV_TAPS = 8;
+__global__ void __launch_bounds__(256) conv_rows_kernel(const __grid_constant__ ConvP p, const float* __restrict__ proj,
+                                                        long long ld, int rows, int pos0,
+                                                        __nv_bfloat16* __restrict__ conv) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 2, t0 = blockIdx.y * CV_ROWS;
+  if (c >= p.C) return;
+  const int t1 = t0 + CV_ROWS < rows ? t0 + CV_ROWS : rows;
+  const float* src = proj + p.off + c;
+  float2 w[CV_TAPS], x[CV_TAPS];   // slot CV_TAPS - 1 is the current token's
+#pragma unroll
+  for (int a = 0; a < CV_TAPS; a++) {
+    const int k = a - (CV_TAPS - p.taps), d = CV_TAPS - 1 - a, q = pos0 + t0 - d;
+    w[a] = k >= 0 ? make_float2(p.w[(size_t)c * p.taps + k], p.w[(size_t)(c + 1) * p.taps + k]) : make_float2(0.f, 0.f);
+    x[a] = make_float2(0.f, 0.f);
+    if (k >= 0 && d > 0 && q >= 0)
+      x[a] = d <= t0 ? *(const float2*)(src + (size_t)(t0 - d) * ld)
+                     : *(const float2*)(p.ring + (size_t)(q % p.taps) * p.C + c);
+  }
+  const float2 b = p.b ? make_float2(p.b[c], p.b[c + 1]) : make_float2(0.f, 0.f);
+#pragma unroll 4
+  for (int t = t0; t < t1; t++) {
+    x[CV_TAPS - 1] = *(const float2*)(src + (size_t)t * ld);
+    float2 y = b;
+#pragma unroll
+    for (int a = 0; a < CV_TAPS; a++) {
+      y.x = fmaf(w[a].x, x[a].x, y.x);
+      y.y = fmaf(w[a].y, x[a].y, y.y);
+    }
+    *(__nv_bfloat162*)(conv + (size_t)t * p.C + c) = __floats2bfloat162_rn(silu_f(y.x), silu_f(y.y));
+#pragma unroll
+    for (int a = 0; a + 1 < CV_TAPS; a++) x[a] = x[a + 1];
+  }
+}
+// step sizes and rates, and for the delta rule the unit-norm factors of (query, key) groups
+__global__ void __launch_bounds__(256) recur_scalars_kernel(const __grid_constant__ RecurP p,
+                                                            const float* __restrict__ proj, long long ld,
+                                                            const __nv_bfloat16* __restrict__ conv,
+                                                            float2* __restrict__ gates, float2* __restrict__ norms) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x, lane = threadIdx.x & 31;
+  const float* row = proj + (size_t)t * ld;
+  for (int h = threadIdx.x; h < p.H; h += blockDim.x) gates[(size_t)t * p.H + h] = recur_gates(p, row, h);
+  if (p.kind != MIX_DELTA) return;
+  for (int g = threadIdx.x >> 5; g < p.G; g += blockDim.x >> 5) {
+    const __nv_bfloat162* q = (const __nv_bfloat162*)(conv + (size_t)t * p.cv.C + p.cq + g * p.D);
+    const __nv_bfloat162* k = (const __nv_bfloat162*)(conv + (size_t)t * p.cv.C + p.ck + g * p.D);
+    float sq = 0.f, sk = 0.f;
+    for (int i = lane; i < p.D / 2; i += 32) {
+      const float2 a = __bfloat1622float2(q[i]), b = __bfloat1622float2(k[i]);
+      sq = fmaf(a.x, a.x, fmaf(a.y, a.y, sq));
+      sk = fmaf(b.x, b.x, fmaf(b.y, b.y, sk));
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0)
+      norms[(size_t)t * p.G + g] = make_float2(rsqrtf(sq + 1e-6f) * rsqrtf((float)p.D), rsqrtf(sk + 1e-6f));
+  }
+}
+
 // after the convolutions of a pass: its last rows become the ring
 __global__ void conv_ring_kernel(const __grid_constant__ ConvP p, const float* __restrict__ proj, long long ld,
                                  int rows, int pos0) {
@@ -375,7 +716,10 @@ __global__ void __launch_bounds__(SC_WARPS * 32) recur_scan_kernel(const __grid_
       const int t = i / CPB, c = i - t * CPB;
       vs[i] = c0 + c < E ? conv[(size_t)(tb + t) * p.cv.C + p.cvv + h * E + c0 + c] : 0.f;
     }
-    if (tid < n) gs[tid] = gates[(size_t)(tb + tid) * p.H + h];
+    if (tid < n) {
+      const float2 gt = gates[(size_t)(tb + tid) * p.H + h];
+      gs[tid] = make_float2(gt.x, decay_of(gt.y));
+    }
     __syncthreads();
     for (int t = 0; t < n; t++) {
       const float2 gt = gs[t];
@@ -427,7 +771,22 @@ __global__ void __launch_bounds__(SC_WARPS * 32) recur_scan_kernel(const __grid_
   }
 }
 
-// delta rule: per-head norm, gate
+__device__ __forceinline__ float4 ld4(const float* p) { return *(const float4*)p; }
+__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
+  const uint2 v = *(const uint2*)p;
+  return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                     __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
+}
+__device__ __forceinline__ float sq4(float4 v, float s) {
+  return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
+}
+
+// delta rule: per-head norm, gate.  One warp per (row, head).
 template <typename OT>
 __global__ void __launch_bounds__(256) delta_finish_kernel(const __grid_constant__ RecurP p, const float* __restrict__ o,
                                                            const float* __restrict__ proj, long long ld,
@@ -435,53 +794,95 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const __grid_constant
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x, lane = threadIdx.x & 31;
+  const bool vec = (p.E & 3) == 0;
   for (int h = threadIdx.x >> 5; h < p.H; h += blockDim.x >> 5) {
     const float* src = o + ((size_t)t * p.H + h) * p.E;
     const float* gate = proj + (size_t)t * ld + p.og + h * p.E;
+    OT* dst = act + (size_t)t * lda + p.oa + h * p.E;
     float sq = 0.f;
-    for (int e = lane; e < p.E; e += 32) sq = fmaf(src[e], src[e], sq);
+    if (vec) {
+      for (int e = lane * 4; e < p.E; e += 128) sq = sq4(ld4(src + e), sq);
+    } else {
+      for (int e = lane; e < p.E; e += 32) sq = fmaf(src[e], src[e], sq);
+    }
     const float r = rsqrtf(warp_sum(sq) / p.E + p.eps) * p.out_scale;
-    for (int e = lane; e < p.E; e += 32)
-      put(act + (size_t)t * lda + p.oa + h * p.E + e, src[e] * r * p.norm[e] * silu_f(gate[e]));
+    if (vec) {
+      for (int e = lane * 4; e < p.E; e += 128) {
+        const float4 v = ld4(src + e), g = ld4(gate + e), w = ld4(p.norm + e);
+        st4(dst + e, make_float4(v.x * r * w.x * silu_f(g.x), v.y * r * w.y * silu_f(g.y), v.z * r * w.z * silu_f(g.z),
+                                 v.w * r * w.w * silu_f(g.w)));
+      }
+    } else {
+      for (int e = lane; e < p.E; e += 32) put(dst + e, src[e] * r * p.norm[e] * silu_f(gate[e]));
+    }
   }
 }
-// ssd: skip, gate, then the norm in equal parts
-template <typename OT>
+// ssd: skip, gate, then the norm in equal parts.  One warp per (row, part); head widths and parts that
+// are multiples of 4 go four at a time, the first SF_HOLD of them held in registers between the passes.
+constexpr int SF_HOLD = 8;
+template <typename OT, typename CT>
 __global__ void __launch_bounds__(256) ssd_finish_kernel(const __grid_constant__ RecurP p, const float* __restrict__ o,
-                                                         const float* __restrict__ conv, const float* __restrict__ proj,
+                                                         const CT* __restrict__ conv, const float* __restrict__ proj,
                                                          long long ld, OT* __restrict__ act, long long lda,
-                                                         int norm_groups) {
-  extern __shared__ __align__(16) float ys[];   // [H * E]
-  __shared__ float red[33];
+                                                         int norm_groups, int rows) {
   pdl_wait();
   pdl_launch_dependents();
-  const int t = blockIdx.x, tid = threadIdx.x, n = p.H * p.E, m = n / norm_groups;
+  const int u = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, t = u / norm_groups;
+  if (t >= rows) return;
+  const int n = p.H * p.E, m = n / norm_groups, i0 = (u - t * norm_groups) * m;
   const float* gate = proj + (size_t)t * ld + p.og;
-  const float* x = conv + (size_t)t * p.cv.C + p.cvv;
-  for (int i = tid; i < n; i += blockDim.x)
-    ys[i] = fmaf(p.Dskip[i / p.E], x[i], o[(size_t)t * n + i]) * silu_f(gate[i]);
-  __syncthreads();
-  for (int g = 0; g < norm_groups; g++) {
-    float sq = 0.f;
-    for (int i = tid; i < m; i += blockDim.x) sq = fmaf(ys[g * m + i], ys[g * m + i], sq);
-    sq = block_sum(sq, red);
-    const float r = rsqrtf(sq / m + p.eps) * p.out_scale;
-    for (int i = tid; i < m; i += blockDim.x)
-      put(act + (size_t)t * lda + p.oa + g * m + i, ys[g * m + i] * r * p.norm[g * m + i]);
+  const CT* x = conv + (size_t)t * p.cv.C + p.cvv;
+  const float* src = o + (size_t)t * n;
+  OT* dst = act + (size_t)t * lda + p.oa;
+  float sq = 0.f;
+  if (((p.E | m) & 3) == 0) {
+    auto y4 = [&](int i) {
+      const float d = p.Dskip[i / p.E];
+      const float4 a = ld4(src + i), b = ld4(x + i), g = ld4(gate + i);
+      return make_float4(fmaf(d, b.x, a.x) * silu_f(g.x), fmaf(d, b.y, a.y) * silu_f(g.y), fmaf(d, b.z, a.z) * silu_f(g.z),
+                         fmaf(d, b.w, a.w) * silu_f(g.w));
+    };
+    float4 v[SF_HOLD];
+#pragma unroll
+    for (int k = 0; k < SF_HOLD; k++) {
+      const int i = lane * 4 + k * 128;
+      v[k] = i < m ? y4(i0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      sq = sq4(v[k], sq);
+    }
+    for (int i = lane * 4 + SF_HOLD * 128; i < m; i += 128) sq = sq4(y4(i0 + i), sq);
+    const float r = rsqrtf(warp_sum(sq) / m + p.eps) * p.out_scale;
+    auto out4 = [&](int i, float4 y) {
+      const float4 w = ld4(p.norm + i);
+      st4(dst + i, make_float4(y.x * r * w.x, y.y * r * w.y, y.z * r * w.z, y.w * r * w.w));
+    };
+#pragma unroll
+    for (int k = 0; k < SF_HOLD; k++) {
+      const int i = lane * 4 + k * 128;
+      if (i < m) out4(i0 + i, v[k]);
+    }
+    for (int i = lane * 4 + SF_HOLD * 128; i < m; i += 128) out4(i0 + i, y4(i0 + i));
+    return;
   }
+  auto y1 = [&](int i) { return fmaf(p.Dskip[i / p.E], to_f(x[i]), src[i]) * silu_f(gate[i]); };
+  for (int i = lane; i < m; i += 32) { const float y = y1(i0 + i); sq = fmaf(y, y, sq); }
+  const float r = rsqrtf(warp_sum(sq) / m + p.eps) * p.out_scale;
+  for (int i = lane; i < m; i += 32) put(dst + i0 + i, y1(i0 + i) * r * p.norm[i0 + i]);
 }
 
-size_t attn_smem(const AttnP& p, int rm) { return (size_t)(rm * (p.Dp + p.Ep + MX_TK + 3) + 40) * sizeof(float); }
-size_t recur_smem(const RecurP& p) { return (size_t)(2 * p.D + 2 * p.E + MX_THREADS + 40) * sizeof(float); }
+size_t attn_smem(const AttnP& p, int rm) {
+  const int fast = p.Dp <= 128 && p.Ep <= 128 ? 8 * rm * p.Ep + 128 : 0;
+  return (size_t)(rm * (p.Dp + p.Ep + MX_TK) + 32 + 40 + p.Dp + p.Ep + fast) * sizeof(float);
+}
+size_t recur_smem(const RecurP& p) { return (size_t)(4 * p.D + 3 * p.E + 2 * MX_THREADS + 40) * sizeof(float); }
 int rm_of(int hpb) { return hpb <= 1 ? 1 : (hpb <= 2 ? 2 : (hpb <= 4 ? 4 : 8)); }
 
-template <typename KT, int RM>
+template <typename KT, int RM, bool FAST>
 int decode_launch(const DecodeArgs& a, int blocks, size_t smem, cudaStream_t s) {
   static std::atomic<unsigned long long> done{0};
-  const int rc = ensure_dynamic_smem(mixers_decode_kernel<KT, RM>, 200 * 1024, done);
+  const int rc = ensure_dynamic_smem(mixers_decode_kernel<KT, RM, FAST>, 200 * 1024, done);
   if (rc) return rc;
   LaunchCfg lc(dim3(blocks), dim3(MX_THREADS), smem, s, pdl_enabled());
-  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, mixers_decode_kernel<KT, RM>, a));
+  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, mixers_decode_kernel<KT, RM, FAST>, a));
   return TLB_OK;
 }
 template <typename KT, int RM>
@@ -522,8 +923,10 @@ int mixers_decode_launch(const AttnP* attn, const RecurP* rec, int n_rec, const 
   DecodeArgs a{};
   int rm = 1;
   size_t smem = 0;
+  bool fast = true;
   if (attn) {
     a.at = *attn;
+    fast = attn->Dp <= 128 && attn->Ep <= 128;
     a.n_attn = attn->G * attn->hb * attn->splits;
     rm = rm_of(attn->hpb);
     smem = attn_smem(*attn, rm);
@@ -539,7 +942,9 @@ int mixers_decode_launch(const AttnP* attn, const RecurP* rec, int n_rec, const 
   a.proj = proj; a.out = out; a.d_pos = d_pos;
 #define MX_CASE(m)                                                                     \
   if (rm == m)                                                                         \
-    return kv_bf16 ? decode_launch<__nv_bfloat16, m>(a, blocks, smem, s) : decode_launch<float, m>(a, blocks, smem, s);
+    return !kv_bf16 ? decode_launch<float, m, false>(a, blocks, smem, s)                  \
+           : fast   ? decode_launch<__nv_bfloat16, m, true>(a, blocks, smem, s)           \
+                    : decode_launch<__nv_bfloat16, m, false>(a, blocks, smem, s);
   MX_CASE(1) MX_CASE(2) MX_CASE(4) MX_CASE(8)
 #undef MX_CASE
   return set_error(TLB_ERR_STATE, "mixers: no head-block width");
@@ -565,11 +970,17 @@ int attn_rows_launch(const AttnP& p, const void* q, const float* proj, long long
   return set_error(TLB_ERR_STATE, "attn_rows: no head-block width");
 }
 
-int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int rows, int pos0, float* conv,
-                           float2* gates, cudaStream_t s) {
-  {
+int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int rows, int pos0, void* conv,
+                           float2* gates, float2* norms, bool chunked, cudaStream_t s) {
+  if (chunked && p.cv.taps > CV_TAPS) return set_error(TLB_ERR_UNSUPPORTED, "recurrent mixer: convolution too long");
+  if (chunked) {
+    LaunchCfg lc(dim3((p.cv.C / 2 + 255) / 256, (rows + CV_ROWS - 1) / CV_ROWS), dim3(256), 0, s, pdl_enabled());
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, conv_rows_kernel, p.cv, proj, ld, rows, pos0, (__nv_bfloat16*)conv));
+    LaunchCfg ls(dim3(rows), dim3(256), 0, s, pdl_enabled());
+    TLB_CUDA(cudaLaunchKernelEx(&ls.cfg, recur_scalars_kernel, p, proj, ld, (const __nv_bfloat16*)conv, gates, norms));
+  } else {
     LaunchCfg lc(dim3(rows), dim3(256), 0, s, pdl_enabled());
-    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, recur_conv_kernel, p, proj, ld, pos0, conv, gates));
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, recur_conv_kernel, p, proj, ld, pos0, (float*)conv, gates));
   }
   if (p.cv.taps > 1) {
     LaunchCfg lc(dim3((p.cv.C + 127) / 128, p.cv.taps - 1), dim3(128), 0, s, pdl_enabled());
@@ -584,25 +995,22 @@ int recur_rows_scan_launch(const RecurP& p, const float* conv, const float2* gat
                              : scan_d<false>(p, conv, gates, o, rows, pos0, s);
 }
 
-int recur_rows_finish_launch(const RecurP& p, const float* o, const float* conv, const float* proj, long long ld,
-                             void* act, long long lda, int norm_groups, int rows, int pos0, bool bf16, cudaStream_t s) {
-  const size_t smem = p.kind == MIX_SSD ? (size_t)p.H * p.E * sizeof(float) : 0;
-  LaunchCfg lc(dim3(rows), dim3(256), smem, s, pdl_enabled());
+int recur_rows_finish_launch(const RecurP& p, const float* o, const void* conv, bool conv_bf16, const float* proj,
+                             long long ld, void* act, long long lda, int norm_groups, int rows, bool bf16, cudaStream_t s) {
+  using B = __nv_bfloat16;
   if (p.kind == MIX_DELTA) {
-    if (bf16) TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, delta_finish_kernel<__nv_bfloat16>, p, o, proj, ld, (__nv_bfloat16*)act, lda));
+    LaunchCfg lc(dim3(rows), dim3(256), 0, s, pdl_enabled());
+    if (bf16) TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, delta_finish_kernel<B>, p, o, proj, ld, (B*)act, lda));
     else TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, delta_finish_kernel<float>, p, o, proj, ld, (float*)act, lda));
     return TLB_OK;
   }
-  static std::atomic<unsigned long long> db{0}, df{0};
-  if (bf16) {
-    const int rc = ensure_dynamic_smem(ssd_finish_kernel<__nv_bfloat16>, 200 * 1024, db);
-    if (rc) return rc;
-    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, ssd_finish_kernel<__nv_bfloat16>, p, o, conv, proj, ld, (__nv_bfloat16*)act, lda, norm_groups));
-  } else {
-    const int rc = ensure_dynamic_smem(ssd_finish_kernel<float>, 200 * 1024, df);
-    if (rc) return rc;
-    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, ssd_finish_kernel<float>, p, o, conv, proj, ld, (float*)act, lda, norm_groups));
-  }
+  LaunchCfg lc(dim3((unsigned)(((long long)rows * norm_groups + 7) / 8)), dim3(256), 0, s, pdl_enabled());
+  if (bf16 && conv_bf16)
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, ssd_finish_kernel<B, B>, p, o, (const B*)conv, proj, ld, (B*)act, lda, norm_groups, rows));
+  else if (bf16)
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, ssd_finish_kernel<B, float>, p, o, (const float*)conv, proj, ld, (B*)act, lda, norm_groups, rows));
+  else
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, ssd_finish_kernel<float, float>, p, o, (const float*)conv, proj, ld, (float*)act, lda, norm_groups, rows));
   return TLB_OK;
 }
 

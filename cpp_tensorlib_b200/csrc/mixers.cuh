@@ -31,7 +31,7 @@ struct AttnP {
   int window, keep, pairs;     // pairs = rotated dimensions / 2
   int oq, ok, ov, og;          // parts of the projected row
   int oa;                      // part of the finished row
-  long long cap, ring;         // cache rows per head = kept slots + ring
+  int cap, ring;               // cache rows per head = kept slots + ring
   float scale, eps, out_scale;
   const float *qn, *kn;
   const float2* inv_freq;      // [pairs] angular frequencies, high and low parts
@@ -107,8 +107,8 @@ __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
 // cache row of position j: the kept first positions have slots of their own
-__device__ __forceinline__ long long kv_slot(const AttnP& p, int j) {
-  return j < p.keep ? j : p.keep + (long long)(j - p.keep) % p.ring;
+__device__ __forceinline__ int kv_slot(const AttnP& p, int j) {
+  return j < p.keep ? j : p.keep + (int)((unsigned)(j - p.keep) % (unsigned)p.ring);
 }
 // What the query at `pos` sees: `kept` first positions, then [lo, pos].
 struct Visible { int kept, lo, n; };
@@ -133,14 +133,18 @@ __device__ __forceinline__ void rot_angle(int pos, float2 f, float* sn, float* c
 }
 
 // one element of a normed and rotated query or key head: src points at the head's raw values, w at
-// its norm weights, rinv is 1 / rms of the whole projection
-__device__ __forceinline__ float rot_elem(const AttnP& p, const float* src, const float* w, float rinv, int pos, int d) {
+// its norm weights, rinv is 1 / rms of the whole projection, cs holds (cos, sin) of the position
+__device__ __forceinline__ float rot_elem(const AttnP& p, const float* src, const float* w, float rinv, const float2* cs,
+                                          int d) {
   if (d >= 2 * p.pairs) return src[d] * rinv * w[d];
   const int e = d & ~1;
   const float u = src[e] * rinv * w[e], v = src[e + 1] * rinv * w[e + 1];
-  float sn, cs;
-  rot_angle(pos, p.inv_freq[d >> 1], &sn, &cs);
-  return (d & 1) ? v * cs + u * sn : u * cs - v * sn;
+  const float2 t = cs[d >> 1];
+  return (d & 1) ? v * t.x + u * t.y : u * t.x - v * t.y;
+}
+constexpr int MX_PAIRS = 512;   // most rotated pairs of a head
+__device__ __forceinline__ void rot_table(const AttnP& p, int pos, float2* cs) {
+  for (int i = threadIdx.x; i < p.pairs; i += blockDim.x) rot_angle(pos, p.inv_freq[i], &cs[i].y, &cs[i].x);
 }
 
 constexpr int MX_THREADS = 256;
@@ -173,7 +177,7 @@ __device__ void attn_range(const AttnP& p, const float* qs, int g, const Visible
 #pragma unroll
       for (int r = 0; r < RM; r++) s[r] = 0.f;
       if (kk < n) {
-        const KT* row = K + kv_slot(p, visible_pos(vis, tb + kk)) * p.Dp;
+        const KT* row = K + (size_t)kv_slot(p, visible_pos(vis, tb + kk)) * p.Dp;
         for (int c = lane & 7; c < p.Dp / CE; c += 8) {
           float f[CE];
           widen16(*(const uint4*)(row + c * CE), f, (const KT*)nullptr);
@@ -220,7 +224,7 @@ __device__ void attn_range(const AttnP& p, const float* qs, int g, const Visible
 #pragma unroll 4
       for (int k = grp; k < n; k += ngrp) {
         float a, b;
-        load2(V + kv_slot(p, visible_pos(vis, tb + k)) * p.Ep + col, a, b);
+        load2(V + (size_t)kv_slot(p, visible_pos(vis, tb + k)) * p.Ep + col, a, b);
 #pragma unroll
         for (int r = 0; r < RM; r++) {
           const float w = sc[r * MX_TK + k];
@@ -261,13 +265,13 @@ __device__ __forceinline__ float conv_silu(const ConvP& p, const float* cur, lon
 // so that hundreds of factors do not add up the exponential's own last-place error.
 __device__ __forceinline__ float decay_of(float x) { return x < 0.5f ? 1.0f + expm1f(-x) : expf(-x); }
 
-// step size and decay of head h: (beta, g) of the delta rule, (dt, decay) of ssd
+// step size and decay rate of head h: (beta, -log g) of the delta rule, (dt, -log decay) of ssd
 __device__ __forceinline__ float2 recur_gates(const RecurP& p, const float* row, int h) {
   if (p.kind == MIX_DELTA)
     return make_float2(sigmoid_f(row[p.ob + h]),
-                       decay_of(expf(p.A_log[h]) * softplus_f(row[p.oa_ + h] + p.dt_bias[h])));
+                       expf(p.A_log[h]) * softplus_f(row[p.oa_ + h] + p.dt_bias[h]));
   const float dt = softplus_f(row[p.ob + h] + p.dt_bias[h]);
-  return make_float2(dt, decay_of(expf(p.A_log[h]) * dt));
+  return make_float2(dt, expf(p.A_log[h]) * dt);
 }
 
 #endif  // __CUDACC__
@@ -279,12 +283,24 @@ int attn_rows_prep_launch(const AttnP& p, const float* proj, long long ld, int r
                           cudaStream_t s);
 int attn_rows_launch(const AttnP& p, const void* q, const float* proj, long long ld, void* act, long long lda, int rows,
                      int pos0, bool bf16, cudaStream_t s);
-int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int rows, int pos0, float* conv,
-                           float2* gates, cudaStream_t s);
+// the same on the tensor pipe (attn_window.cu): bf16, widths up to 128
+bool attn_window_eligible(const AttnP& p);
+int attn_window_launch(const AttnP& p, const void* q, const float* proj, long long ld, void* act, long long lda,
+                       int rows, int pos0, cudaStream_t s);
+// Convolutions, step sizes and rates of a pass, in one of two forms: f32 with the delta rule's unit
+// queries and keys (norms NULL), for the token-by-token scan; or bf16 as the convolutions leave them,
+// with the factors that make queries and keys unit vectors apart ([rows][G] query, key), for the chunks.
+int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int rows, int pos0, void* conv,
+                           float2* gates, float2* norms, bool chunked, cudaStream_t s);
 int recur_rows_scan_launch(const RecurP& p, const float* conv, const float2* gates, float* o, int rows, int pos0,
                            cudaStream_t s);
-int recur_rows_finish_launch(const RecurP& p, const float* o, const float* conv, const float* proj, long long ld,
-                             void* act, long long lda, int norm_groups, int rows, int pos0, bool bf16, cudaStream_t s);
+int recur_rows_finish_launch(const RecurP& p, const float* o, const void* conv, bool conv_bf16, const float* proj,
+                             long long ld, void* act, long long lda, int norm_groups, int rows, bool bf16, cudaStream_t s);
+// the recurrence in chunks on the tensor pipe (recur_chunk.cu)
+bool recur_chunk_eligible(const RecurP& p);
+size_t recur_chunk_scratch_bytes(const RecurP& p, int rows);
+int recur_chunk_launch(const RecurP& p, const void* conv, const float2* gates, const float2* norms, void* scratch,
+                       float* o, int rows, int pos0, cudaStream_t s);
 int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, long long ldo, int n, float eps, int rows,
                     bool bf16, cudaStream_t s);
 int embed_scaled_launch(const void* embed, const int* ids, float* x, int width, long long ld, float scale, int rows,

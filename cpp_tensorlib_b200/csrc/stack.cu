@@ -60,9 +60,9 @@ struct StackDecoder : DecoderBase {
   float *x = nullptr, *proj = nullptr, *act = nullptr, *mb = nullptr;
   // prompt pass: rows of pf_rows tokens (hr, actr and ffr in the product's operand type)
   int pf_rows = 0;
-  float *xr = nullptr, *projr = nullptr, *convr = nullptr, *orr = nullptr, *tmpr = nullptr, *gath = nullptr;
-  float2* gater = nullptr;
-  void *hr = nullptr, *qr = nullptr, *actr = nullptr, *ffr = nullptr, *hg = nullptr;
+  float *xr = nullptr, *projr = nullptr, *orr = nullptr, *tmpr = nullptr, *gath = nullptr;
+  float2 *gater = nullptr, *normr = nullptr;
+  void *convr = nullptr, *chunkr = nullptr, *hr = nullptr, *qr = nullptr, *actr = nullptr, *ffr = nullptr, *hg = nullptr;
   int* idx = nullptr;
   std::vector<void*> pf_owned;
 
@@ -159,6 +159,14 @@ int StackDecoder::prefill_begin(int rows, cudaStream_t s) {
   get(&convr, R * conv_max * 4);
   get(&orr, R * o_max * 4);
   get(&gater, R * gate_max * sizeof(float2));
+  get(&normr, R * gate_max * sizeof(float2));
+  size_t cb = 0;
+  for (auto& L : layers)
+    for (int i = 0; i < L.n_rec; i++) {
+      const size_t n = bf16 && recur_chunk_eligible(L.rec[i]) ? recur_chunk_scratch_bytes(L.rec[i], rows) : 0;
+      cb = n > cb ? n : cb;
+    }
+  get(&chunkr, cb);
   get(&gath, R * hidden * 4);
   get(&hr, R * pad8(hidden) * es());
   get(&hg, R * pad8(hidden) * es());
@@ -192,13 +200,18 @@ int StackDecoder::prefill_pass(const int* d_ids, int rows, int pos, cudaStream_t
     PF(product(c, hr, E8, L.in, projr, L.proj_n, false, rows, s));
     if (L.has_attn) {
       PF(attn_rows_prep_launch(L.at, projr, L.proj_n, rows, pos, qr, bf16, s));
-      PF(attn_rows_launch(L.at, qr, projr, L.proj_n, actr, L.act_n, rows, pos, bf16, s));
+      if (bf16 && attn_window_eligible(L.at))
+        PF(attn_window_launch(L.at, qr, projr, L.proj_n, actr, L.act_n, rows, pos, s));
+      else
+        PF(attn_rows_launch(L.at, qr, projr, L.proj_n, actr, L.act_n, rows, pos, bf16, s));
     }
     for (int i = 0; i < L.n_rec; i++) {
       const RecurP& r = L.rec[i];
-      PF(recur_rows_conv_launch(r, projr, L.proj_n, rows, pos, convr, gater, s));
-      PF(recur_rows_scan_launch(r, convr, gater, orr, rows, pos, s));
-      PF(recur_rows_finish_launch(r, orr, convr, projr, L.proj_n, actr, L.act_n, L.norm_groups[i], rows, pos, bf16, s));
+      const bool chunks = bf16 && recur_chunk_eligible(r);
+      PF(recur_rows_conv_launch(r, projr, L.proj_n, rows, pos, convr, gater, normr, chunks, s));
+      if (chunks) PF(recur_chunk_launch(r, convr, gater, normr, chunkr, orr, rows, pos, s));
+      else PF(recur_rows_scan_launch(r, (const float*)convr, gater, orr, rows, pos, s));
+      PF(recur_rows_finish_launch(r, orr, convr, chunks, projr, L.proj_n, actr, L.act_n, L.norm_groups[i], rows, bf16, s));
     }
     PF(product(c, actr, L.act_n, L.out, xr, hidden, true, rows, s));
     if (!L.ff) continue;
