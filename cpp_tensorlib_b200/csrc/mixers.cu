@@ -51,23 +51,49 @@ __device__ __forceinline__ AttnUnit attn_unit_of(const AttnP& p, int unit, int p
   a.t1 = a.t0 + chunk < a.vis.n ? a.t0 + chunk : a.vis.n;
   return a;
 }
+// sum of squares of n values of the projected row, this thread's share, 16 values in flight
+__device__ __forceinline__ float row_squares(const float* x, int n) {
+  float s = 0.f;
+  if ((n & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < n; i += 16 * MX_THREADS) {
+      float4 v[4];
+#pragma unroll
+      for (int k = 0; k < 4; k++)
+        v[k] = i + k * 4 * MX_THREADS < n ? *(const float4*)(x + i + k * 4 * MX_THREADS) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < 4; k++) s = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, s))));
+    }
+  } else {
+    for (int i = threadIdx.x; i < n; i += MX_THREADS) s = fmaf(x[i], x[i], s);
+  }
+  return s;
+}
+// norm weights of the unit's heads, before the projected row is there: wn [RM][Dp] | [Dp]
+template <int RM>
+__device__ void attn_norm_weights(const AttnP& p, const AttnUnit& a, float* wn) {
+  for (int i = threadIdx.x; i < (RM + 1) * p.Dp; i += MX_THREADS) {
+    const int r = i / p.Dp, d = i - r * p.Dp;
+    float v = 0.f;
+    if (d < p.D && r < a.nh) v = p.qn[(a.h0 + r) * p.D + d];
+    if (d < p.D && r == RM) v = p.kn[a.g * p.D + d];
+    wn[i] = v;
+  }
+}
 // normed and rotated query heads of the unit into qs [RM][Dp]; with the range that ends with the token
-// itself, its key and value into the cache and (bf16 values) into knew [Dp] | [Ep]
+// itself, its key and value into the cache and (in the cache's type) into knew [Dp] | [Ep]
 template <typename KT, int RM>
 __device__ void attn_token_heads(const AttnP& p, const AttnUnit& a, const float* row, int pos, const float2* cs,
-                                 float* qs, KT* knew, float* red) {
+                                 const float* wn, float* qs, KT* knew, float* red) {
   const int tid = threadIdx.x;
   const bool last = a.split == a.active - 1;
-  float sq = 0.f, sk = 0.f;
-  for (int i = tid; i < p.H * p.D; i += MX_THREADS) { const float v = row[p.oq + i]; sq = fmaf(v, v, sq); }
-  if (last)
-    for (int i = tid; i < p.G * p.D; i += MX_THREADS) { const float v = row[p.ok + i]; sk = fmaf(v, v, sk); }
+  float sq = row_squares(row + p.oq, p.H * p.D);
+  float sk = last ? row_squares(row + p.ok, p.G * p.D) : 0.f;
   sq = block_sum(sq, red);
   const float rq = rsqrtf(sq / (p.H * p.D) + p.eps);
   for (int i = tid; i < RM * p.Dp; i += MX_THREADS) {
     const int r = i / p.Dp, d = i - r * p.Dp;
     float v = 0.f;
-    if (r < a.nh && d < p.D) v = rot_elem(p, row + p.oq + (a.h0 + r) * p.D, p.qn + (a.h0 + r) * p.D, rq, cs, d);
+    if (r < a.nh && d < p.D) v = rot_elem(p, row + p.oq + (a.h0 + r) * p.D, wn + r * p.Dp, rq, cs, d);
     if (sizeof(KT) == 2) v = __bfloat162float(__float2bfloat16_rn(v));
     qs[i] = v;
   }
@@ -78,7 +104,7 @@ __device__ void attn_token_heads(const AttnP& p, const AttnUnit& a, const float*
     KT* kd = (KT*)p.K + ((size_t)a.g * p.cap + slot) * p.Dp;
     KT* vd = (KT*)p.V + ((size_t)a.g * p.cap + slot) * p.Ep;
     for (int d = tid; d < p.Dp; d += MX_THREADS) {
-      const float v = d < p.D ? rot_elem(p, row + p.ok + a.g * p.D, p.kn + a.g * p.D, rk, cs, d) : 0.f;
+      const float v = d < p.D ? rot_elem(p, row + p.ok + a.g * p.D, wn + RM * p.Dp, rk, cs, d) : 0.f;
       put(kd + d, v);
       put(knew + d, v);
     }
@@ -91,72 +117,78 @@ __device__ void attn_token_heads(const AttnP& p, const AttnUnit& a, const float*
   __syncthreads();
 }
 
-template <int RM>
-__device__ void attn_finish(const AttnP& p, const float* os, const float* ml, int h0, int nh, const float* row,
-                            float* out) {
-  for (int i = threadIdx.x; i < nh * p.E; i += MX_THREADS) {
-    const int r = i / p.E, e = i - r * p.E, c = (h0 + r) * p.E + e;
-    out[p.oa + c] = os[r * p.Ep + e] / ml[RM + r] * sigmoid_f(row[p.og + c]) * p.out_scale;
-  }
-}
-// a range's unnormalised heads (os), maxima and sums (ml) into the partials; the last range to arrive
-// merges them all
+// A range's unnormalised heads (os), maxima and sums (ml) into the partials; the last range to arrive
+// merges them all and applies the output gate.  Partials of a unit: [splits][hpb][Ep], then
+// [splits][hpb] (maximum, sum).
 template <int RM>
 __device__ void attn_merge(const AttnP& p, const AttnUnit& a, float* os, float* ml, float* sc, const float* row,
                            float* out) {
   __shared__ int s_last;
   const int tid = threadIdx.x, nh = a.nh, active = a.active;
-  if (active == 1) {
-    attn_finish<RM>(p, os, ml, a.h0, nh, row, out);
-    return;
-  }
-  const int PS = p.Ep + 2;
-  float* part = p.part + (size_t)a.gb * p.splits * p.hpb * PS;
-  for (int i = tid; i < nh * p.Ep; i += MX_THREADS)
-    part[((size_t)a.split * p.hpb + i / p.Ep) * PS + i % p.Ep] = os[i];
-  if (tid < nh) {
-    part[((size_t)a.split * p.hpb + tid) * PS + p.Ep] = ml[tid];
-    part[((size_t)a.split * p.hpb + tid) * PS + p.Ep + 1] = ml[RM + tid];
-  }
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) s_last = atomicAdd(&p.counters[a.gb], 1) == active - 1;
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
-  if (tid == 0) p.counters[a.gb] = 0;
-  const int warp = tid >> 5, lane = tid & 31;
-  for (int r = warp; r < nh; r += MX_THREADS / 32) {
-    float m = -3.0e38f;
-    for (int s = lane; s < active; s += 32) m = fmaxf(m, __ldcg(&part[((size_t)s * p.hpb + r) * PS + p.Ep]));
-    m = warp_max(m);
-    float l = 0.f;
-    for (int s = lane; s < active; s += 32) {
-      const float w = expf(__ldcg(&part[((size_t)s * p.hpb + r) * PS + p.Ep]) - m);
-      sc[r * MX_TK + s] = w;
-      l = fmaf(w, __ldcg(&part[((size_t)s * p.hpb + r) * PS + p.Ep + 1]), l);
-    }
-    l = warp_sum(l);
-    if (lane == 0) ml[RM + r] = l;
-  }
-  __syncthreads();
-  for (int i = tid; i < nh * p.Ep; i += MX_THREADS) {
-    const int r = i / p.Ep, e = i - r * p.Ep;
-    const float* src = part + (size_t)r * PS + e;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    int s = 0;
-    for (; s + 8 <= active; s += 8) {
-      float v[8];
+  constexpr int GH = 4;
+  float gate[GH];   // of the first GH elements this thread finishes
 #pragma unroll
-      for (int k = 0; k < 8; k++) v[k] = __ldcg(src + (size_t)(s + k) * p.hpb * PS);
-#pragma unroll
-      for (int k = 0; k < 8; k++) acc[k & 3] = fmaf(sc[r * MX_TK + s + k], v[k], acc[k & 3]);
-    }
-    for (; s < active; s++) acc[0] = fmaf(sc[r * MX_TK + s], __ldcg(src + (size_t)s * p.hpb * PS), acc[0]);
-    os[i] = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+  for (int k = 0; k < GH; k++) {
+    const int i = tid + k * MX_THREADS;
+    gate[k] = i < nh * p.E ? row[p.og + a.h0 * p.E + i] : 0.f;
   }
-  __syncthreads();
-  attn_finish<RM>(p, os, ml, a.h0, nh, row, out);
+  if (active > 1) {
+    const int slots = p.splits * p.hpb;
+    float* part = p.part + (size_t)a.gb * attn_part_floats(p);
+    float2* stat = (float2*)(part + (size_t)slots * p.Ep);
+    for (int i = tid; i < nh * p.Ep / 4; i += MX_THREADS)
+      ((float4*)(part + (size_t)a.split * p.hpb * p.Ep))[i] = ((const float4*)os)[i];
+    if (tid < nh) stat[a.split * p.hpb + tid] = make_float2(ml[tid], ml[RM + tid]);
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) s_last = atomicAdd(&p.counters[a.gb], 1) == active - 1;
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    if (tid == 0) p.counters[a.gb] = 0;
+    const int warp = tid >> 5, lane = tid & 31;
+    for (int r = warp; r < nh; r += MX_THREADS / 32) {
+      float m = -3.0e38f;
+      for (int s = lane; s < active; s += 32) m = fmaxf(m, __ldcg(&stat[s * p.hpb + r]).x);
+      m = warp_max(m);
+      float l = 0.f;
+      for (int s = lane; s < active; s += 32) {
+        const float2 v = __ldcg(&stat[s * p.hpb + r]);
+        const float w = expf(v.x - m);
+        sc[r * MX_TK + s] = w;
+        l = fmaf(w, v.y, l);
+      }
+      l = warp_sum(l);
+      if (lane == 0) ml[RM + r] = l;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * p.Ep / 4; i += MX_THREADS) {
+      const int r = i * 4 / p.Ep;
+      const float4* src = (const float4*)part + i;
+      const size_t step = (size_t)p.hpb * p.Ep / 4;
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int s0 = 0; s0 < active; s0 += 12) {
+        float4 v[12];
+#pragma unroll
+        for (int k = 0; k < 12; k++)
+          v[k] = s0 + k < active ? __ldcg(src + (size_t)(s0 + k) * step) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int k = 0; k < 12; k++) {
+          const float w = s0 + k < active ? sc[r * MX_TK + s0 + k] : 0.f;
+          acc.x = fmaf(w, v[k].x, acc.x); acc.y = fmaf(w, v[k].y, acc.y);
+          acc.z = fmaf(w, v[k].z, acc.z); acc.w = fmaf(w, v[k].w, acc.w);
+        }
+      }
+      ((float4*)os)[i] = acc;
+    }
+    __syncthreads();
+  }
+  for (int i = tid, k = 0; i < nh * p.E; i += MX_THREADS, k++) {
+    const int r = i / p.E, e = i - r * p.E, c = a.h0 * p.E + i;
+    float g = k == 0 ? gate[0] : (k == 1 ? gate[1] : (k == 2 ? gate[2] : gate[3]));
+    if (k >= GH) g = row[p.og + c];
+    out[p.oa + c] = os[r * p.Ep + e] / ml[RM + r] * sigmoid_f(g) * p.out_scale;
+  }
 }
 
 // any widths, either cache type
@@ -168,14 +200,16 @@ __device__ void attn_decode_unit(const AttnP& p, int unit, const float* row, flo
   float* sc = os + RM * p.Ep;             // [RM][MX_TK]
   float* ml = sc + RM * MX_TK;            // [3][RM], 32
   float* red = ml + 32;                   // [33], 40
-  KT* knew = (KT*)(red + 40);             // [Dp + Ep]
+  float* wn = red + 40;                   // [RM + 1][Dp]
+  KT* knew = (KT*)(wn + (RM + 1) * p.Dp); // [Dp + Ep]
   const AttnUnit a = attn_unit_of(p, unit, pos);
   if (a.split >= a.active) { pdl_wait(); return; }
   rot_table(p, pos, cs);
+  attn_norm_weights<RM>(p, a, wn);
   pdl_wait();
   pdl_launch_dependents();
   __syncthreads();
-  attn_token_heads<KT, RM>(p, a, row, pos, cs, qs, knew, red);
+  attn_token_heads<KT, RM>(p, a, row, pos, cs, wn, qs, knew, red);
   attn_range<KT, RM>(p, qs, a.g, a.vis, a.t0, a.t1, sc, os, ml);
   attn_merge<RM>(p, a, os, ml, sc, row, out);
 }
@@ -217,7 +251,8 @@ __device__ void attn_decode_unit16(const AttnP& p, int unit, const float* row, f
   float* sc = os + RM * p.Ep;             // [RM][MX_TK]
   float* ml = sc + RM * MX_TK;            // [3][RM], 32
   float* red = ml + 32;                   // [33], 40
-  KT* knew = (KT*)(red + 40);             // [Dp + Ep]
+  float* wn = red + 40;                   // [RM + 1][Dp]
+  KT* knew = (KT*)(wn + (RM + 1) * p.Dp); // [Dp + Ep]
   float* wo = (float*)(knew + 256);       // [8 warps][RM][Ep]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, ch = tid & 15, kr = tid >> 4;
   const AttnUnit a = attn_unit_of(p, unit, pos);
@@ -237,11 +272,12 @@ __device__ void attn_decode_unit16(const AttnP& p, int unit, const float* row, f
   load(kf, K, p.Dp, ck, a.t0);
   load(vf, V, p.Ep, cv, a.t0);
   rot_table(p, pos, cs);
+  attn_norm_weights<RM>(p, a, wn);
   pdl_wait();
   pdl_launch_dependents();
   if (tid < RM) { ml[tid] = -3.0e38f; ml[RM + tid] = 0.f; }
   __syncthreads();
-  attn_token_heads<KT, RM>(p, a, row, pos, cs, qs, knew, red);
+  attn_token_heads<KT, RM>(p, a, row, pos, cs, wn, qs, knew, red);
   float acc[RM][8];
 #pragma unroll
   for (int r = 0; r < RM; r++)
@@ -374,21 +410,48 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
     return i < D ? p.cq + kg * D + i : (i < 2 * D ? p.ck + kg * D + i - D : p.cvv + h * E + i - 2 * D);
   };
   const int taps = p.cv.taps;
-  for (int i = tid; i < n; i += MX_THREADS) {
-    const int c = channel(i);
-    const float* w = p.cv.w + (size_t)c * taps;
-    float y = p.cv.b ? p.cv.b[c] : 0.f;
-    for (int a = 0; a + 1 < taps; a++) {
-      const int qp = pos - (taps - 1 - a);
-      if (qp >= 0) y = fmaf(w[a], p.cv.ring[(size_t)(qp % taps) * p.cv.C + c], y);
+  const float A_log = p.A_log[h], bias = p.dt_bias[h], skip = p.kind == MIX_SSD ? p.Dskip[h] : 0.f;
+  const float nw = p.kind == MIX_DELTA && tid < E ? p.norm[tid] : 0.f;
+  for (int i0 = 0; i0 < n; i0 += 2 * MX_THREADS) {
+    // two channels a thread, four taps at a time: every load of the history before its first use
+    float y[2] = {0.f, 0.f};
+    for (int a0 = 0; a0 + 1 < taps; a0 += 4) {
+      float w[2][4], x[2][4];
+      int at = (pos - (taps - 1 - a0) + taps) % taps;   // ring row of tap a0 (not read in front of the start)
+      if (at < 0) at += taps;
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        const bool on = a0 + j + 1 < taps && pos - (taps - 1 - a0 - j) >= 0;
+#pragma unroll
+        for (int b = 0; b < 2; b++) {
+          const int i = i0 + b * MX_THREADS + tid;
+          const int c = i < n ? channel(i) : 0;
+          w[b][j] = on && i < n ? p.cv.w[(size_t)c * taps + a0 + j] : 0.f;
+          x[b][j] = on && i < n ? p.cv.ring[(size_t)at * p.cv.C + c] : 0.f;
+        }
+        at = at + 1 == taps ? 0 : at + 1;
+      }
+#pragma unroll
+      for (int j = 0; j < 4; j++) {
+        y[0] = fmaf(w[0][j], x[0][j], y[0]);
+        y[1] = fmaf(w[1][j], x[1][j], y[1]);
+      }
     }
-    sm[i] = y;
-    wl[i] = w[taps - 1];
+#pragma unroll
+    for (int b = 0; b < 2; b++) {
+      const int i = i0 + b * MX_THREADS + tid;
+      if (i < n) {
+        const int c = channel(i);
+        sm[i] = p.cv.b ? y[b] + p.cv.b[c] : y[b];
+        wl[i] = p.cv.w[(size_t)c * taps + taps - 1];
+      }
+    }
   }
-  const float rate = expf(p.A_log[h]), bias = p.dt_bias[h];
   pdl_wait();
   pdl_launch_dependents();
   const float* cur = row + p.cv.off;
+  const float gate = tid < E ? row[p.og + h * E + tid] : 0.f;
+  const float raw_in = row[p.ob + h], raw_step = row[p.oa_ + h];
   for (int i = tid; i < n; i += MX_THREADS) {
     const int c = channel(i);
     const float x = cur[c];
@@ -396,8 +459,8 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
     if (taps > 1 && (i >= 2 * D || h == kg * rep)) p.cv.ring[(size_t)(pos % taps) * p.cv.C + c] = x;
   }
   const bool delta = p.kind == MIX_DELTA;
-  const float step = softplus_f(row[p.oa_ + h] + bias);
-  const float in = delta ? sigmoid_f(row[p.ob + h]) : step, g = decay_of(rate * step);
+  const float step = softplus_f(raw_step + bias);
+  const float in = delta ? sigmoid_f(raw_in) : step, g = decay_of(expf(A_log) * step);
   __syncthreads();
   if (delta) {
     float sq = 0.f, sk = 0.f;
@@ -484,10 +547,11 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
     for (int e = tid; e < E; e += MX_THREADS) sq = fmaf(o[e], o[e], sq);
     sq = block_sum(sq, rs);
     const float r = rsqrtf(sq / E + p.eps) * p.out_scale;
-    for (int e = tid; e < E; e += MX_THREADS) out[p.oa + h * E + e] = o[e] * r * p.norm[e] * silu_f(row[p.og + h * E + e]);
+    for (int e = tid; e < E; e += MX_THREADS)
+      out[p.oa + h * E + e] = o[e] * r * (e == tid ? nw : p.norm[e]) * silu_f(e == tid ? gate : row[p.og + h * E + e]);
   } else {
     for (int e = tid; e < E; e += MX_THREADS)
-      out[p.oa + h * E + e] = fmaf(p.Dskip[h], v[e], o[e]) * silu_f(row[p.og + h * E + e]);
+      out[p.oa + h * E + e] = fmaf(skip, v[e], o[e]) * silu_f(e == tid ? gate : row[p.og + h * E + e]);
   }
 }
 
@@ -871,7 +935,7 @@ __global__ void __launch_bounds__(256) ssd_finish_kernel(const __grid_constant__
 
 size_t attn_smem(const AttnP& p, int rm) {
   const int fast = p.Dp <= 128 && p.Ep <= 128 ? 8 * rm * p.Ep + 128 : 0;
-  return (size_t)(rm * (p.Dp + p.Ep + MX_TK) + 32 + 40 + p.Dp + p.Ep + fast) * sizeof(float);
+  return (size_t)(rm * (2 * p.Dp + p.Ep + MX_TK) + 32 + 40 + 2 * p.Dp + p.Ep + fast) * sizeof(float);
 }
 size_t recur_smem(const RecurP& p) { return (size_t)(4 * p.D + 3 * p.E + 2 * MX_THREADS + 40) * sizeof(float); }
 int rm_of(int hpb) { return hpb <= 1 ? 1 : (hpb <= 2 ? 2 : (hpb <= 4 ? 4 : 8)); }

@@ -37,9 +37,14 @@ struct AttnP {
   const float2* inv_freq;      // [pairs] angular frequencies, high and low parts
   void *K, *V;                 // [G][cap][Dp], [G][cap][Ep]
   int splits, hb, hpb;         // key ranges of a token, head blocks of a group, heads per block
-  float* part;                 // [G*hb][splits][hpb][E + 2]
+  float* part;                 // [G*hb] x ([splits][hpb][Ep] | [splits][hpb] (max, sum))
   int* counters;               // [G*hb]
 };
+
+// floats of one unit's partials (a multiple of 4: units start on 16 bytes)
+__host__ __device__ inline size_t attn_part_floats(const AttnP& p) {
+  return ((size_t)p.splits * p.hpb * (p.Ep + 2) + 3) & ~(size_t)3;
+}
 
 struct ConvP {
   const float *w, *b;          // [C][taps], [C] or NULL

@@ -298,7 +298,7 @@ static int build(StackDecoder* d, const tlb_stack_cfg* cfg, const tlb_layer_cfg*
         p.splits = max_i(1, (2 * c->sm_count) / units);
         if (p.splits > (most + 63) / 64) p.splits = (most + 63) / 64;
         if (p.splits > MX_TK) p.splits = MX_TK;
-        if (!rc) rc = d->alloc((void**)&p.part, (size_t)units * p.splits * p.hpb * (p.Ep + 2) * 4, d->owned);
+        if (!rc) rc = d->alloc((void**)&p.part, units * attn_part_floats(p) * 4, d->owned);
         if (!rc) rc = d->alloc((void**)&p.counters, (size_t)units * sizeof(int), d->owned);
         std::vector<float2> f(max_i(1, p.pairs));
         for (int i = 0; i < p.pairs; i++) {
