@@ -2,9 +2,12 @@
 // RMS norm (whole row, or a segment in equal parts) on the staged activation in front, a residual
 // add or the clipped gated unit behind.  W is bf16 or f32 row-major, everything else f32.
 //
-// HBM bound.  A warp owns one row, or two adjacent rows (gate and up interleaved), and keeps eight
-// 16-byte loads in flight plus the next eight; the first eight are issued BEFORE the wait for the
-// preceding kernel, so a launch's weight stream starts under its predecessor's tail.
+// HBM bound.  A stream of ks adjacent warps owns one row, or two adjacent rows (gate and up
+// interleaved), each warp its own part of K; ks is picked on the host so that the streams of all SMs
+// come out even.  Every warp keeps eight 16-byte loads in flight plus the next eight; the first eight
+// are issued BEFORE the wait for the preceding kernel, so a launch's weight stream starts under its
+// predecessor's tail.  Weights are marked evict-first in the L2: a token streams gigabytes of them
+// once, and what every launch needs again -- instructions, states, activations -- should stay.
 #include "mixers.cuh"
 
 namespace tlb {
@@ -13,22 +16,92 @@ namespace {
 
 constexpr int RG_WARPS = 8;
 
-__device__ __forceinline__ uint4 rg_ld(const void* p) {
+__device__ __forceinline__ uint4 rg_ld(const void* p, uint64_t pol) {
   uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];"
-               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  asm volatile("ld.global.nc.L1::no_allocate.L2::cache_hint.v4.u32 {%0,%1,%2,%3}, [%4], %5;"
+               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p), "l"(pol));
   return v;
 }
 
+// x into xs [ldw], zero behind K; eight 16-byte loads in flight a thread
+__device__ __forceinline__ void rg_stage(const RowGemv& p, float* xs) {
+  if ((uintptr_t)p.x & 15) {   // a row of a width that is no multiple of 4
+    for (int i = threadIdx.x; i < p.ldw; i += RG_WARPS * 32) xs[i] = i < p.K ? p.x[i] : 0.f;
+    return;
+  }
+  const int n4 = (int)(p.ldw / 4), k4 = p.K / 4;   // ldw is a multiple of 8
+  for (int i0 = threadIdx.x; i0 < n4; i0 += 8 * RG_WARPS * 32) {
+    float4 v[8];
+#pragma unroll
+    for (int u = 0; u < 8; u++) {
+      const int i = i0 + u * RG_WARPS * 32;
+      v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < k4) v[u] = ((const float4*)p.x)[i];
+      else if (i == k4 && i < n4) {
+        const int r = p.K - 4 * k4;
+        if (r > 0) v[u].x = p.x[4 * i];
+        if (r > 1) v[u].y = p.x[4 * i + 1];
+        if (r > 2) v[u].z = p.x[4 * i + 2];
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 8; u++) {
+      const int i = i0 + u * RG_WARPS * 32;
+      if (i < n4) ((float4*)xs)[i] = v[u];
+    }
+  }
+}
+
+// the norm in place: one part by the whole block, several parts a warp each
+__device__ __forceinline__ void rg_norm(const RowGemv& p, float* xs, float* red) {
+  const int tid = threadIdx.x, lane = tid & 31, m = p.n_len / p.n_groups;
+  if (p.n_groups == 1) {
+    float* seg = xs + p.n_off;
+    float sq = 0.f;
+    for (int i = tid; i < m; i += RG_WARPS * 32) sq = fmaf(seg[i], seg[i], sq);
+    sq = block_sum(sq, red);
+    const float s = rsqrtf(sq / m + p.eps) * p.nscale;
+#pragma unroll 8
+    for (int i = tid; i < m; i += RG_WARPS * 32) seg[i] = seg[i] * s * p.nw[i];
+    return;
+  }
+  for (int g = tid >> 5; g < p.n_groups; g += RG_WARPS) {
+    float* seg = xs + p.n_off + g * m;
+    float sq = 0.f;
+#pragma unroll 8
+    for (int i = lane; i < m; i += 32) sq = fmaf(seg[i], seg[i], sq);
+    const float s = rsqrtf(warp_sum(sq) / m + p.eps) * p.nscale;
+#pragma unroll 8
+    for (int i = lane; i < m; i += 32) seg[i] = seg[i] * s * p.nw[g * m + i];
+  }
+}
+
+template <int R>
+__device__ __forceinline__ void rg_emit(const RowGemv& p, int rg, const float (&a)[R]) {
+  if (p.epi == 2) {
+    if (R == 2) p.y[rg] = glu_clipped(a[0], a[R - 1], p.limit);
+    return;
+  }
+#pragma unroll
+  for (int r = 0; r < R; r++) {
+    const int n = rg * R + r;
+    if (n < p.N) p.y[n] = p.epi == 1 ? p.y[n] + a[r] : a[r];
+  }
+}
+
 template <typename WT, int R>
-__global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid_constant__ RowGemv p) {
+__global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid_constant__ RowGemv p, int ks) {
   constexpr int CE = Vec16<WT>::N, U = 8 / R;
-  extern __shared__ __align__(16) float xs[];   // [ldw], zero behind K
+  extern __shared__ __align__(16) float xs[];   // [ldw], then the streams' partial sums
   __shared__ float red[33];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int chunks = (int)(p.ldw / CE), groups = (p.N + R - 1) / R, stride = gridDim.x * RG_WARPS;
+  const int groups = (p.N + R - 1) / R, ns = RG_WARPS / ks, stream = warp / ks, sub = warp - stream * ks;
+  const int stride = gridDim.x * ns, chunks = (int)(p.ldw / CE), per = (chunks + ks - 1) / ks;
+  const int c_lo = sub * per, c_hi = c_lo + per < chunks ? c_lo + per : chunks;
+  float* part = xs + p.ldw;                     // [local group][stream][R][ks]
   const WT* W = (const WT*)p.W;
-  int rg = blockIdx.x * RG_WARPS + warp, cb = 0;
+  const uint64_t pol = l2_evict_first_policy();
+  int rg = blockIdx.x * ns + stream, cb = c_lo, loc = 0;
   uint4 cur[R][U], nxt[R][U];
   auto fetch = [&](uint4 (&w)[R][U], int g, int b) {
 #pragma unroll
@@ -37,38 +110,32 @@ __global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid
 #pragma unroll
       for (int u = 0; u < U; u++) {
         const int c = b + lane + 32 * u;
-        w[r][u] = c < chunks ? rg_ld(row + (size_t)c * CE) : make_uint4(0, 0, 0, 0);
+        w[r][u] = c < c_hi ? rg_ld(row + (size_t)c * CE, pol) : make_uint4(0, 0, 0, 0);
       }
     }
   };
-  if (rg < groups) fetch(cur, rg, 0);
+  if (rg < groups) fetch(cur, rg, cb);
+  if (p.nw)   // the norm's weights into the L2
+    for (int i = tid * 32; i < p.n_len; i += RG_WARPS * 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.nw + i));
   pdl_wait();
   pdl_launch_dependents();
-  for (int i = tid; i < p.ldw; i += RG_WARPS * 32) xs[i] = i < p.K ? p.x[i] : 0.f;
-  if (p.nw) {
-    const int m = p.n_len / p.n_groups;
-    for (int g = 0; g < p.n_groups; g++) {
-      float* seg = xs + p.n_off + g * m;
-      float sq = 0.f;
-      __syncthreads();
-      for (int i = tid; i < m; i += RG_WARPS * 32) sq = fmaf(seg[i], seg[i], sq);
-      sq = block_sum(sq, red);
-      const float s = rsqrtf(sq / m + p.eps) * p.nscale;
-      for (int i = tid; i < m; i += RG_WARPS * 32) seg[i] = seg[i] * s * p.nw[g * m + i];
-    }
-  }
+  rg_stage(p, xs);
   __syncthreads();
+  if (p.nw) {
+    rg_norm(p, xs, red);
+    __syncthreads();
+  }
   float acc[R][2];
 #pragma unroll
   for (int r = 0; r < R; r++) acc[r][0] = acc[r][1] = 0.f;
   while (rg < groups) {
     int ng = rg, nb = cb + 32 * U;
-    if (nb >= chunks) { ng += stride; nb = 0; }
+    if (nb >= c_hi) { ng += stride; nb = c_lo; }
     if (ng < groups) fetch(nxt, ng, nb);
 #pragma unroll
     for (int u = 0; u < U; u++) {
       const int c = cb + lane + 32 * u;
-      if (c < chunks) {
+      if (c < c_hi) {
         float x[CE];
 #pragma unroll
         for (int e = 0; e < CE; e += 4) {
@@ -92,16 +159,14 @@ __global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid
         acc[r][0] = acc[r][1] = 0.f;
       }
       if (lane == 0) {
-        if (p.epi == 2) {
-          if (R == 2) p.y[rg] = glu_clipped(a[0], a[R - 1], p.limit);
+        if (ks == 1) {
+          rg_emit<R>(p, rg, a);
         } else {
 #pragma unroll
-          for (int r = 0; r < R; r++) {
-            const int n = rg * R + r;
-            if (n < p.N) p.y[n] = p.epi == 1 ? p.y[n] + a[r] : a[r];
-          }
+          for (int r = 0; r < R; r++) part[((loc * ns + stream) * R + r) * ks + sub] = a[r];
         }
       }
+      loc++;
     }
     rg = ng;
     cb = nb;
@@ -110,6 +175,20 @@ __global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid
 #pragma unroll
       for (int u = 0; u < U; u++) cur[r][u] = nxt[r][u];
   }
+  if (ks == 1) return;
+  __syncthreads();
+  for (int i = tid;; i += RG_WARPS * 32) {
+    const int l = i / ns, g = (blockIdx.x * ns + i - l * ns) + l * stride;
+    if (l * stride + (int)blockIdx.x * ns >= groups) break;
+    if (g >= groups) continue;
+    float a[R];
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+      a[r] = 0.f;
+      for (int k = 0; k < ks; k++) a[r] += part[(i * R + r) * ks + k];
+    }
+    rg_emit<R>(p, g, a);
+  }
 }
 
 template <typename WT, int R>
@@ -117,10 +196,22 @@ int rg_launch(DeviceCtx* c, const RowGemv& p, cudaStream_t s) {
   static std::atomic<unsigned long long> done{0};
   const int rc = ensure_dynamic_smem(row_gemv_kernel<WT, R>, 220 * 1024, done);
   if (rc) return rc;
-  const int need = ((p.N + R - 1) / R + RG_WARPS - 1) / RG_WARPS;
-  const int ctas = need < 2 * c->sm_count ? need : 2 * c->sm_count;
-  LaunchCfg lc(dim3(ctas), dim3(RG_WARPS * 32), (size_t)p.ldw * sizeof(float), s, pdl_enabled());
-  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, row_gemv_kernel<WT, R>, p));
+  const int groups = (p.N + R - 1) / R, chunks = (int)(p.ldw / Vec16<WT>::N), full = 2 * c->sm_count;
+  // warps a stream: the fewest that come within 3 % of the most even division, each with a batch to load
+  int ks = 1;
+  double best = 1e30;
+  for (int k = 1; k <= RG_WARPS; k *= 2) {
+    if (k > 1 && chunks / k < 32 * 4) break;
+    const int ns = RG_WARPS / k;
+    const double cost = (double)((groups + full * ns - 1) / (full * ns)) / k;
+    if (cost < best * 0.97) { best = cost; ks = k; }
+  }
+  const int ns = RG_WARPS / ks, need = (groups + ns - 1) / ns, ctas = need < full ? need : full;
+  const int local = (groups + ctas * ns - 1) / (ctas * ns);
+  const size_t smem = ((size_t)p.ldw + (ks > 1 ? (size_t)local * ns * R * ks : 0)) * sizeof(float);
+  if (smem > 220 * 1024) return set_error(TLB_ERR_UNSUPPORTED, "row_gemv: the activation row does not fit the shared-memory stage");
+  LaunchCfg lc(dim3(ctas), dim3(RG_WARPS * 32), smem, s, pdl_enabled());
+  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, row_gemv_kernel<WT, R>, p, ks));
   return TLB_OK;
 }
 
@@ -141,13 +232,18 @@ __global__ void __launch_bounds__(256) rms_rows_kernel(const float* __restrict__
   for (int i = threadIdx.x; i < n; i += 256) put(dst + i, row[i] * r * w[i]);
 }
 
+// 1024 columns a block
 template <typename WT>
 __global__ void embed_scaled_kernel(const WT* __restrict__ embed, long long ld, const int* __restrict__ ids,
                                     float* __restrict__ x, int width, float scale) {
   pdl_wait();
   pdl_launch_dependents();
   const WT* src = embed + (size_t)ids[blockIdx.x] * ld;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) x[(size_t)blockIdx.x * width + i] = to_f(src[i]) * scale;
+#pragma unroll
+  for (int k = 0; k < 4; k++) {
+    const int i = blockIdx.y * 1024 + k * 256 + threadIdx.x;
+    if (i < width) x[(size_t)blockIdx.x * width + i] = to_f(src[i]) * scale;
+  }
 }
 
 __global__ void gather_rows_kernel(const float* __restrict__ x, const int* __restrict__ idx, float* __restrict__ out,
@@ -170,9 +266,7 @@ __global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict_
 }  // namespace
 
 int row_gemv_launch(DeviceCtx* c, const RowGemv& p, bool bf16, cudaStream_t s) {
-  if (p.ldw * (long long)sizeof(float) > 216 * 1024)
-    return set_error(TLB_ERR_UNSUPPORTED, "row_gemv: the activation row does not fit the shared-memory stage");
-  // two rows a warp where the rows come in pairs, or where there are enough of them to fill the SMs
+  // two rows a stream where the rows come in pairs, or where there are enough of them to fill the SMs
   const bool two = p.epi == 2 || p.N >= 2 * 2 * c->sm_count * RG_WARPS;
   if (bf16) return two ? rg_launch<__nv_bfloat16, 2>(c, p, s) : rg_launch<__nv_bfloat16, 1>(c, p, s);
   return two ? rg_launch<float, 2>(c, p, s) : rg_launch<float, 1>(c, p, s);
@@ -188,7 +282,7 @@ int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, lo
 
 int embed_scaled_launch(const void* embed, const int* ids, float* x, int width, long long ld, float scale, int rows,
                         bool bf16, cudaStream_t s) {
-  LaunchCfg lc(dim3(rows), dim3(256), 0, s, pdl_enabled());
+  LaunchCfg lc(dim3(rows, (width + 1023) / 1024), dim3(256), 0, s, pdl_enabled());
   if (bf16) TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, embed_scaled_kernel<__nv_bfloat16>, (const __nv_bfloat16*)embed, ld, ids, x, width, scale));
   else TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, embed_scaled_kernel<float>, (const float*)embed, ld, ids, x, width, scale));
   return TLB_OK;

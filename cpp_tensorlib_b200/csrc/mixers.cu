@@ -664,9 +664,9 @@ __global__ void __launch_bounds__(256) recur_conv_kernel(const __grid_constant__
   for (int h = threadIdx.x; h < p.H; h += blockDim.x) gates[(size_t)t * p.H + h] = recur_gates(p, row, h);
 }
 
-// The same for the chunked form: a thread runs down CT rows of two adjacent channels with the last
+// The same for the chunked form: a thread runs down CV_ROWS rows of two adjacent channels with the last
 // inputs in registers.
-constexpr int CV_ROWS = 32, CV_TAPS = 8;
+constexpr int CV_ROWS = 32, CV_TAPS = 8, CV_STEP = 8;
 __global__ void __launch_bounds__(256) conv_rows_kernel(const __grid_constant__ ConvP p, const float* __restrict__ proj,
                                                         long long ld, int rows, int pos0,
                                                         __nv_bfloat16* __restrict__ conv) {
@@ -676,29 +676,35 @@ __global__ void __launch_bounds__(256) conv_rows_kernel(const __grid_constant__ 
   if (c >= p.C) return;
   const int t1 = t0 + CV_ROWS < rows ? t0 + CV_ROWS : rows;
   const float* src = proj + p.off + c;
-  float2 w[CV_TAPS], x[CV_TAPS];   // slot CV_TAPS - 1 is the current token's
+  float2 w[CV_TAPS], x[CV_TAPS - 1 + CV_STEP];   // x: the last inputs, then those of CV_STEP rows
 #pragma unroll
   for (int a = 0; a < CV_TAPS; a++) {
     const int k = a - (CV_TAPS - p.taps), d = CV_TAPS - 1 - a, q = pos0 + t0 - d;
     w[a] = k >= 0 ? make_float2(p.w[(size_t)c * p.taps + k], p.w[(size_t)(c + 1) * p.taps + k]) : make_float2(0.f, 0.f);
+    if (d == 0) continue;
     x[a] = make_float2(0.f, 0.f);
-    if (k >= 0 && d > 0 && q >= 0)
+    if (k >= 0 && q >= 0)
       x[a] = d <= t0 ? *(const float2*)(src + (size_t)(t0 - d) * ld)
                      : *(const float2*)(p.ring + (size_t)(q % p.taps) * p.C + c);
   }
   const float2 b = p.b ? make_float2(p.b[c], p.b[c + 1]) : make_float2(0.f, 0.f);
-#pragma unroll 4
-  for (int t = t0; t < t1; t++) {
-    x[CV_TAPS - 1] = *(const float2*)(src + (size_t)t * ld);
-    float2 y = b;
+  for (int t = t0; t < t1; t += CV_STEP) {
 #pragma unroll
-    for (int a = 0; a < CV_TAPS; a++) {
-      y.x = fmaf(w[a].x, x[a].x, y.x);
-      y.y = fmaf(w[a].y, x[a].y, y.y);
+    for (int i = 0; i < CV_STEP; i++)
+      x[CV_TAPS - 1 + i] = t + i < t1 ? *(const float2*)(src + (size_t)(t + i) * ld) : make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < CV_STEP; i++) {
+      float2 y = b;
+#pragma unroll
+      for (int a = 0; a < CV_TAPS; a++) {
+        y.x = fmaf(w[a].x, x[a + i].x, y.x);
+        y.y = fmaf(w[a].y, x[a + i].y, y.y);
+      }
+      if (t + i < t1)
+        *(__nv_bfloat162*)(conv + (size_t)(t + i) * p.C + c) = __floats2bfloat162_rn(silu_f(y.x), silu_f(y.y));
     }
-    *(__nv_bfloat162*)(conv + (size_t)t * p.C + c) = __floats2bfloat162_rn(silu_f(y.x), silu_f(y.y));
 #pragma unroll
-    for (int a = 0; a + 1 < CV_TAPS; a++) x[a] = x[a + 1];
+    for (int a = 0; a + 1 < CV_TAPS; a++) x[a] = x[a + CV_STEP];
   }
 }
 // step sizes and rates, and for the delta rule the unit-norm factors of (query, key) groups
