@@ -23,56 +23,52 @@ __device__ __forceinline__ uint4 rg_ld(const void* p, uint64_t pol) {
   return v;
 }
 
-// x into xs [ldw], zero behind K; eight 16-byte loads in flight a thread
-__device__ __forceinline__ void rg_stage(const RowGemv& p, float* xs) {
-  if ((uintptr_t)p.x & 15) {   // a row of a width that is no multiple of 4
-    for (int i = threadIdx.x; i < p.ldw; i += RG_WARPS * 32) xs[i] = i < p.K ? p.x[i] : 0.f;
-    return;
-  }
-  const int n4 = (int)(p.ldw / 4), k4 = p.K / 4;   // ldw is a multiple of 8
-  for (int i0 = threadIdx.x; i0 < n4; i0 += 8 * RG_WARPS * 32) {
-    float4 v[8];
+// x into xs [ldw], zero behind K; returns this thread's share of its sum of squares.  Kept short: a
+// launch runs this code once, from a cold instruction cache.
+__device__ __forceinline__ float rg_stage(const RowGemv& p, float* xs) {
+  float sq = 0.f;
+  const int k4 = ((uintptr_t)p.x & 15) ? 0 : p.K / 4;   // rows of an odd width go one by one
+  for (int i0 = threadIdx.x; i0 < k4; i0 += 4 * RG_WARPS * 32) {
+    float4 v[4];
 #pragma unroll
-    for (int u = 0; u < 8; u++) {
-      const int i = i0 + u * RG_WARPS * 32;
-      v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i < k4) v[u] = ((const float4*)p.x)[i];
-      else if (i == k4 && i < n4) {
-        const int r = p.K - 4 * k4;
-        if (r > 0) v[u].x = p.x[4 * i];
-        if (r > 1) v[u].y = p.x[4 * i + 1];
-        if (r > 2) v[u].z = p.x[4 * i + 2];
+    for (int u = 0; u < 4; u++)
+      if (i0 + u * RG_WARPS * 32 < k4) v[u] = ((const float4*)p.x)[i0 + u * RG_WARPS * 32];
+#pragma unroll
+    for (int u = 0; u < 4; u++)
+      if (i0 + u * RG_WARPS * 32 < k4) {
+        ((float4*)xs)[i0 + u * RG_WARPS * 32] = v[u];
+        sq = fmaf(v[u].x, v[u].x, fmaf(v[u].y, v[u].y, fmaf(v[u].z, v[u].z, fmaf(v[u].w, v[u].w, sq))));
       }
-    }
-#pragma unroll
-    for (int u = 0; u < 8; u++) {
-      const int i = i0 + u * RG_WARPS * 32;
-      if (i < n4) ((float4*)xs)[i] = v[u];
-    }
   }
+#pragma unroll 1
+  for (int i = 4 * k4 + threadIdx.x; i < p.ldw; i += RG_WARPS * 32) {
+    const float x = i < p.K ? p.x[i] : 0.f;
+    xs[i] = x;
+    sq = fmaf(x, x, sq);
+  }
+  return sq;
 }
 
-// the norm in place: one part by the whole block, several parts a warp each
-__device__ __forceinline__ void rg_norm(const RowGemv& p, float* xs, float* red) {
-  const int tid = threadIdx.x, lane = tid & 31, m = p.n_len / p.n_groups;
-  if (p.n_groups == 1) {
-    float* seg = xs + p.n_off;
-    float sq = 0.f;
-    for (int i = tid; i < m; i += RG_WARPS * 32) sq = fmaf(seg[i], seg[i], sq);
-    sq = block_sum(sq, red);
-    const float s = rsqrtf(sq / m + p.eps) * p.nscale;
-#pragma unroll 8
-    for (int i = tid; i < m; i += RG_WARPS * 32) seg[i] = seg[i] * s * p.nw[i];
+// the norm in place: the whole row by the block, a segment in parts a warp each
+__device__ __forceinline__ void rg_norm(const RowGemv& p, float* xs, float sq, float* red) {
+  const int tid = threadIdx.x, lane = tid & 31;
+  if (p.n_groups == 1 && p.n_len == p.K) {
+    const float s = rsqrtf(block_sum(sq, red) / p.K + p.eps) * p.nscale;
+#pragma unroll 4
+    for (int i = tid; i < p.K; i += RG_WARPS * 32) xs[i] *= s * p.nw[i];
     return;
   }
+  __syncthreads();
+  const int m = p.n_len / p.n_groups;
+#pragma unroll 1
   for (int g = tid >> 5; g < p.n_groups; g += RG_WARPS) {
     float* seg = xs + p.n_off + g * m;
-    float sq = 0.f;
-#pragma unroll 8
-    for (int i = lane; i < m; i += 32) sq = fmaf(seg[i], seg[i], sq);
-    const float s = rsqrtf(warp_sum(sq) / m + p.eps) * p.nscale;
-#pragma unroll 8
-    for (int i = lane; i < m; i += 32) seg[i] = seg[i] * s * p.nw[g * m + i];
+    float q = 0.f;
+#pragma unroll 4
+    for (int i = lane; i < m; i += 32) q = fmaf(seg[i], seg[i], q);
+    const float s = rsqrtf(warp_sum(q) / m + p.eps) * p.nscale;
+#pragma unroll 4
+    for (int i = lane; i < m; i += 32) seg[i] *= s * p.nw[g * m + i];
   }
 }
 
@@ -119,12 +115,9 @@ __global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid
     for (int i = tid * 32; i < p.n_len; i += RG_WARPS * 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.nw + i));
   pdl_wait();
   pdl_launch_dependents();
-  rg_stage(p, xs);
+  const float sq = rg_stage(p, xs);
+  if (p.nw) rg_norm(p, xs, sq, red);
   __syncthreads();
-  if (p.nw) {
-    rg_norm(p, xs, red);
-    __syncthreads();
-  }
   float acc[R][2];
 #pragma unroll
   for (int r = 0; r < R; r++) acc[r][0] = acc[r][1] = 0.f;
@@ -197,7 +190,7 @@ int rg_launch(DeviceCtx* c, const RowGemv& p, cudaStream_t s) {
   const int rc = ensure_dynamic_smem(row_gemv_kernel<WT, R>, 220 * 1024, done);
   if (rc) return rc;
   const int groups = (p.N + R - 1) / R, chunks = (int)(p.ldw / Vec16<WT>::N), full = 2 * c->sm_count;
-  // warps a stream: the fewest that come within 3 % of the most even division, each with a batch to load
+  // warps a stream (single rows): the fewest that come within 3 % of the most even division
   int ks = 1;
   double best = 1e30;
   for (int k = 1; k <= RG_WARPS; k *= 2) {
@@ -205,6 +198,7 @@ int rg_launch(DeviceCtx* c, const RowGemv& p, cudaStream_t s) {
     const int ns = RG_WARPS / k;
     const double cost = (double)((groups + full * ns - 1) / (full * ns)) / k;
     if (cost < best * 0.97) { best = cost; ks = k; }
+    if (R == 2) break;   // two rows a warp: the extra sums cost more than the unevenness
   }
   const int ns = RG_WARPS / ks, need = (groups + ns - 1) / ns, ctas = need < full ? need : full;
   const int local = (groups + ctas * ns - 1) / (ctas * ns);
