@@ -6,8 +6,9 @@
 // convolutions, the state update and the read-out, and finishes the head.
 //
 // Prompt pass: row-batched launches.  attn_rows_prep (norm, rotation, cache rows), attn_rows
-// (attention of every row), recur_rows_conv (convolutions, unit norms, step sizes and decays),
-// recur_rows_scan (the recurrence, state in registers), recur_rows_finish (norms and gates).
+// (attention of every row), recur_rows_conv (convolutions, unit norms, step sizes and decay rates),
+// recur_rows_scan (the recurrence, state in registers), recur_rows_finish (norms and gates).  bf16
+// models take attn_window.cu and recur_chunk.cu for attention and recurrence where the widths allow.
 #include "mixers.cuh"
 
 namespace tlb {
