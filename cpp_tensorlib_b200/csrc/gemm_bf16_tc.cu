@@ -3,6 +3,8 @@
 //   EPI 0  C[m,n]  = acc                      (f32)
 //   EPI 1  C[m,n] += acc                      (f32 residual)
 //   EPI 2  O[m,j]  = glu(acc[2j], acc[2j+1])  (bf16, gate and up rows interleaved in W)
+//   EPI 3  O[m,n]  = acc                      (bf16)
+//   EPI 4  O[m,n]  = relu(acc)^2              (bf16)
 //
 // Persistent: one CTA per SM walks the 128 x BN output tiles.  Warp 0 is the TMA producer of both
 // operands (64-k stages, 128-byte swizzle, boxes past M, N or K read as zeros), warp 1 issues
@@ -195,6 +197,28 @@ __global__ void __launch_bounds__(GT_THREADS, 1)
                 o[j] = __float2bfloat16_rn(
                     glu_clipped(__uint_as_float(v[2 * j]), __uint_as_float(v[2 * j + 1]), p.limit));
           }
+        } else if (EPI >= 3) {
+          __nv_bfloat16* o = p.O + (long long)m * p.ldo + n0 + c0;
+          if (EPI == 4) {
+#pragma unroll
+            for (int j = 0; j < 32; j++) v[j] = __float_as_uint(relu2(__uint_as_float(v[j])));
+          }
+          if (n0 + c0 + 32 <= p.N && (p.ldo & 7) == 0) {
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+              uint32_t w[4];
+#pragma unroll
+              for (int k = 0; k < 4; k++) {
+                const __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(v[8 * j + 2 * k]), __uint_as_float(v[8 * j + 2 * k + 1]));
+                w[k] = *(const uint32_t*)&h;
+              }
+              ((uint4*)o)[j] = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 32; j++)
+              if (n0 + c0 + j < p.N) o[j] = __float2bfloat16_rn(__uint_as_float(v[j]));
+          }
         } else {
           float* o = p.C + (long long)m * p.ldc + n0 + c0;
           if (n0 + c0 + 32 <= p.N && (p.ldc & 3) == 0) {
@@ -273,9 +297,13 @@ int gemm_bf16_tc_launch(DeviceCtx* c, const void* a, long long lda, const void* 
   if (rc) return rc;
   GtParams p{C, ldc, (__nv_bfloat16*)O, ldo, M, N, K, mt, (N + BN - 1) / BN, limit, c->status};
 #define GT_CASE(bn)                                                            \
-  if (BN == bn)                                                                \
-    return epi == 0 ? gt_launch<bn, 0>(c, ta, tb, p, s)                        \
-                    : (epi == 1 ? gt_launch<bn, 1>(c, ta, tb, p, s) : gt_launch<bn, 2>(c, ta, tb, p, s));
+  if (BN == bn) switch (epi) {                                                 \
+      case 0: return gt_launch<bn, 0>(c, ta, tb, p, s);                        \
+      case 1: return gt_launch<bn, 1>(c, ta, tb, p, s);                        \
+      case 2: return gt_launch<bn, 2>(c, ta, tb, p, s);                        \
+      case 3: return gt_launch<bn, 3>(c, ta, tb, p, s);                        \
+      default: return gt_launch<bn, 4>(c, ta, tb, p, s);                       \
+    }
   GT_CASE(256) GT_CASE(128) GT_CASE(64) GT_CASE(32)
 #undef GT_CASE
   return set_error(TLB_ERR_STATE, "gemm_bf16_tc: no tile width");

@@ -1,6 +1,7 @@
-// One-row matrix product of the layer-stack decoder, y = W . f(x), with its neighbours fused: an
-// RMS norm (whole row, or a segment in equal parts) on the staged activation in front, a residual
-// add or the clipped gated unit behind.  W is bf16 or f32 row-major, everything else f32.
+// One-row matrix product of the layer-stack decoder, y = W . f(x), with its neighbours fused: on the
+// staged activation in front, the residual sum that a norm of the preceding sublayer's output ends in,
+// an RMS norm (whole row, or a segment in equal parts) and a silu gate; a residual add, the clipped
+// gated unit or the square of relu behind.  W is bf16 or f32 row-major, everything else f32.
 //
 // HBM bound.  A stream of ks adjacent warps owns one row, or two adjacent rows (gate and up
 // interleaved), each warp its own part of K; ks is picked on the host so that the streams of all SMs
@@ -49,13 +50,28 @@ __device__ __forceinline__ float rg_stage(const RowGemv& p, float* xs) {
   return sq;
 }
 
+// the preceding sublayer's output, normed, added to the residual: every block computes the row, block 0
+// leaves it for the launches behind.  Returns the thread's share of the new row's sum of squares.
+__device__ __forceinline__ float rg_residual(const RowGemv& p, float* xs, float sq, float* red) {
+  const float s = rsqrtf(block_sum(sq, red) / p.K + p.eps);
+  sq = 0.f;
+#pragma unroll 8
+  for (int i = threadIdx.x; i < p.K; i += RG_WARPS * 32) {
+    const float v = fmaf(xs[i] * s, p.rn[i], p.res[i]);
+    xs[i] = v;
+    if (p.xout && blockIdx.x == 0) p.xout[i] = v;
+    sq = fmaf(v, v, sq);
+  }
+  return sq;
+}
+
 // the norm in place: the whole row by the block, a segment in parts a warp each
 __device__ __forceinline__ void rg_norm(const RowGemv& p, float* xs, float sq, float* red) {
   const int tid = threadIdx.x, lane = tid & 31;
   if (p.n_groups == 1 && p.n_len == p.K) {
     const float s = rsqrtf(block_sum(sq, red) / p.K + p.eps) * p.nscale;
 #pragma unroll 4
-    for (int i = tid; i < p.K; i += RG_WARPS * 32) xs[i] *= s * p.nw[i];
+    for (int i = tid; i < p.K; i += RG_WARPS * 32) xs[i] *= p.gate ? s * p.nw[i] * silu_f(p.gate[i]) : s * p.nw[i];
     return;
   }
   __syncthreads();
@@ -68,7 +84,8 @@ __device__ __forceinline__ void rg_norm(const RowGemv& p, float* xs, float sq, f
     for (int i = lane; i < m; i += 32) q = fmaf(seg[i], seg[i], q);
     const float s = rsqrtf(warp_sum(q) / m + p.eps) * p.nscale;
 #pragma unroll 4
-    for (int i = lane; i < m; i += 32) seg[i] *= s * p.nw[g * m + i];
+    for (int i = lane; i < m; i += 32)
+      seg[i] *= p.gate ? s * p.nw[g * m + i] * silu_f(p.gate[g * m + i]) : s * p.nw[g * m + i];
   }
 }
 
@@ -81,7 +98,7 @@ __device__ __forceinline__ void rg_emit(const RowGemv& p, int rg, const float (&
 #pragma unroll
   for (int r = 0; r < R; r++) {
     const int n = rg * R + r;
-    if (n < p.N) p.y[n] = p.epi == 1 ? p.y[n] + a[r] : a[r];
+    if (n < p.N) p.y[n] = p.epi == 1 ? p.y[n] + a[r] : (p.epi == 3 ? relu2(a[r]) : a[r]);
   }
 }
 
@@ -113,9 +130,12 @@ __global__ void __launch_bounds__(RG_WARPS * 32, 2) row_gemv_kernel(const __grid
   if (rg < groups) fetch(cur, rg, cb);
   if (p.nw)   // the norm's weights into the L2
     for (int i = tid * 32; i < p.n_len; i += RG_WARPS * 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.nw + i));
+  if (p.rn)
+    for (int i = tid * 32; i < p.K; i += RG_WARPS * 32 * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.rn + i));
   pdl_wait();
   pdl_launch_dependents();
-  const float sq = rg_stage(p, xs);
+  float sq = rg_stage(p, xs);
+  if (p.res) sq = rg_residual(p, xs, sq, red);
   if (p.nw) rg_norm(p, xs, sq, red);
   __syncthreads();
   float acc[R][2];
@@ -213,7 +233,7 @@ int rg_launch(DeviceCtx* c, const RowGemv& p, cudaStream_t s) {
 template <typename OT>
 __global__ void __launch_bounds__(256) rms_rows_kernel(const float* __restrict__ x, long long ldx,
                                                        const float* __restrict__ w, OT* __restrict__ out, long long ldo,
-                                                       int n, float eps) {
+                                                       int n, float eps, float scale) {
   __shared__ float red[33];
   pdl_wait();
   pdl_launch_dependents();
@@ -222,8 +242,50 @@ __global__ void __launch_bounds__(256) rms_rows_kernel(const float* __restrict__
   float sq = 0.f;
   for (int i = threadIdx.x; i < n; i += 256) sq = fmaf(row[i], row[i], sq);
   sq = block_sum(sq, red);
-  const float r = rsqrtf(sq / n + eps);
+  const float r = rsqrtf(sq / n + eps) * scale;
   for (int i = threadIdx.x; i < n; i += 256) put(dst + i, row[i] * r * w[i]);
+}
+
+// x += norm(y) * w, the sum also as the next product's operand; without y only the latter
+constexpr int RR_HOLD = 8;    // values of y a thread keeps between the passes
+template <typename OT>
+__global__ void __launch_bounds__(512) residual_rows_kernel(float* __restrict__ x, const float* __restrict__ y,
+                                                            const float* __restrict__ w, OT* __restrict__ out,
+                                                            long long ldo, int n, float eps) {
+  __shared__ float red[33];
+  pdl_wait();
+  pdl_launch_dependents();
+  float* row = x + (size_t)blockIdx.x * n;
+  OT* dst = out + (size_t)blockIdx.x * ldo;
+  if (!y) {
+    for (int i = threadIdx.x; i < n; i += 512) put(dst + i, row[i]);
+    return;
+  }
+  const float* yr = y + (size_t)blockIdx.x * n;
+  float v[RR_HOLD], sq = 0.f;
+#pragma unroll
+  for (int k = 0; k < RR_HOLD; k++) {
+    const int i = threadIdx.x + k * 512;
+    v[k] = i < n ? yr[i] : 0.f;
+    sq = fmaf(v[k], v[k], sq);
+  }
+  for (int i = threadIdx.x + RR_HOLD * 512; i < n; i += 512) sq = fmaf(yr[i], yr[i], sq);
+  sq = block_sum(sq, red);
+  const float r = rsqrtf(sq / n + eps);
+#pragma unroll
+  for (int k = 0; k < RR_HOLD; k++) {
+    const int i = threadIdx.x + k * 512;
+    if (i < n) {
+      const float s = fmaf(v[k] * r, w[i], row[i]);
+      row[i] = s;
+      put(dst + i, s);
+    }
+  }
+  for (int i = threadIdx.x + RR_HOLD * 512; i < n; i += 512) {
+    const float s = fmaf(yr[i] * r, w[i], row[i]);
+    row[i] = s;
+    put(dst + i, s);
+  }
 }
 
 // 1024 columns a block
@@ -257,6 +319,13 @@ __global__ void glu_rows_kernel(const float* __restrict__ gu, float* __restrict_
   }
 }
 
+__global__ void relu2_rows_kernel(const float* __restrict__ u, float* __restrict__ out, long long n) {
+  pdl_wait();
+  pdl_launch_dependents();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    out[i] = relu2(u[i]);
+}
+
 }  // namespace
 
 int row_gemv_launch(DeviceCtx* c, const RowGemv& p, bool bf16, cudaStream_t s) {
@@ -266,11 +335,30 @@ int row_gemv_launch(DeviceCtx* c, const RowGemv& p, bool bf16, cudaStream_t s) {
   return two ? rg_launch<float, 2>(c, p, s) : rg_launch<float, 1>(c, p, s);
 }
 
-int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, long long ldo, int n, float eps, int rows,
-                    bool bf16, cudaStream_t s) {
+int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, long long ldo, int n, float eps,
+                    float scale, int rows, bool bf16, cudaStream_t s) {
   LaunchCfg lc(dim3(rows), dim3(256), 0, s, pdl_enabled());
-  if (bf16) TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, rms_rows_kernel<__nv_bfloat16>, x, ldx, w, (__nv_bfloat16*)out, ldo, n, eps));
-  else TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, rms_rows_kernel<float>, x, ldx, w, (float*)out, ldo, n, eps));
+  if (bf16)
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, rms_rows_kernel<__nv_bfloat16>, x, ldx, w, (__nv_bfloat16*)out, ldo, n, eps, scale));
+  else
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, rms_rows_kernel<float>, x, ldx, w, (float*)out, ldo, n, eps, scale));
+  return TLB_OK;
+}
+
+int residual_rows_launch(float* x, const float* y, const float* w, void* out, long long ldo, int n, float eps, int rows,
+                         bool bf16, cudaStream_t s) {
+  LaunchCfg lc(dim3(rows), dim3(512), 0, s, pdl_enabled());
+  if (bf16)
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, residual_rows_kernel<__nv_bfloat16>, x, y, w, (__nv_bfloat16*)out, ldo, n, eps));
+  else
+    TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, residual_rows_kernel<float>, x, y, w, (float*)out, ldo, n, eps));
+  return TLB_OK;
+}
+
+int relu2_rows_launch(const float* u, float* out, int ff, int rows, cudaStream_t s) {
+  const long long n = (long long)rows * ff, b = (n + 255) / 256;
+  LaunchCfg lc(dim3((unsigned)(b < 148 * 16 ? b : 148 * 16)), dim3(256), 0, s, pdl_enabled());
+  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, relu2_rows_kernel, u, out, n));
   return TLB_OK;
 }
 

@@ -3,7 +3,9 @@
 // One token: ONE launch for all mixers of a layer.  Blocks are divided among them by index: the
 // attention takes (key/value head, head block, key range) units whose last arriver merges the
 // ranges and applies the output gate; a recurrent mixer takes one block per head, which runs the
-// convolutions, the state update and the read-out, and finishes the head.
+// convolutions, the state update and the read-out, and finishes the head -- except gla, which has no
+// convolution and takes a block per 32 state columns (norm and gate follow with the output projection).
+// Latent attention has launches of its own (attn_latent.cu).
 //
 // Prompt pass: row-batched launches.  attn_rows_prep (norm, rotation, cache rows), attn_rows
 // (attention of every row), recur_rows_conv (convolutions, unit norms, step sizes and decay rates),
@@ -556,6 +558,75 @@ __device__ void recur_decode_head(const RecurP& p, int h, const float* row, floa
   }
 }
 
+// ---- gated linear attention, one token ------------------------------------------------------
+// One block per (head, 32 state columns): warp w holds rows w, w + 8, ... of them.  The state and the
+// decay's weights are fetched before the projected row is there.
+constexpr int GL_COLS = 32, GL_WARPS = MX_THREADS / 32, GL_PRE = 16;
+__device__ __forceinline__ int gla_slices(const RecurP& p) { return (p.E + GL_COLS - 1) / GL_COLS; }
+__device__ void gla_decode_unit(const RecurP& p, int unit, const float* row, float* out, int pos, float* sm) {
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, D = p.D, E = p.E;
+  const int nsl = gla_slices(p), h = unit / nsl, e = (unit - h * nsl) * GL_COLS + lane, HD = p.H * D;
+  float* q = sm;               // [D]
+  float* k = q + D;            // [D]
+  float* al = k + D;           // [D]
+  float* red = al + D;         // [GL_WARPS][32]
+  float* S = p.S + (size_t)h * D * E + e;
+  const bool on = e < E;
+  float s[MX_ROWS], w[GL_PRE];
+  auto fetch = [&](int d0) {
+#pragma unroll
+    for (int i = 0; i < MX_ROWS; i++) {
+      const int d = d0 + warp + i * GL_WARPS;
+      s[i] = on && pos > 0 && d < D ? S[(size_t)d * E] : 0.f;
+    }
+  };
+  fetch(0);
+  const int c0 = h * D + tid;
+#pragma unroll
+  for (int r = 0; r < GL_PRE; r++) w[r] = tid < D && r < p.rank ? p.a_up[(size_t)r * HD + c0] : 0.f;
+  const float b0 = tid < D ? p.a_bias[c0] : 0.f;
+  pdl_wait();
+  pdl_launch_dependents();
+  const float v = on ? row[p.cvv + h * E + e] : 0.f;
+  for (int d = tid; d < D; d += MX_THREADS) {
+    const int c = h * D + d;
+    q[d] = row[p.cq + c] * rsqrtf((float)D);
+    k[d] = row[p.ck + c];
+    float z = d == tid ? b0 : p.a_bias[c];
+#pragma unroll
+    for (int r = 0; r < GL_PRE; r++)
+      if (r < p.rank) z = fmaf(row[p.ob + r], d == tid ? w[r] : p.a_up[(size_t)r * HD + c], z);
+    for (int r = GL_PRE; r < p.rank; r++) z = fmaf(row[p.ob + r], p.a_up[(size_t)r * HD + c], z);
+    al[d] = decay_of(gla_rate(z, p.tau));
+  }
+  __syncthreads();
+  float acc = 0.f;
+  for (int d0 = 0; d0 < D; d0 += GL_WARPS * MX_ROWS) {
+    if (d0) fetch(d0);
+#pragma unroll
+    for (int i = 0; i < MX_ROWS; i++) {
+      const int d = d0 + warp + i * GL_WARPS;
+      if (d < D) {
+        s[i] = fmaf(k[d], v, s[i] * al[d]);
+        acc = fmaf(q[d], s[i], acc);
+        if (on) S[(size_t)d * E] = s[i];
+      }
+    }
+  }
+  red[tid] = acc;
+  __syncthreads();
+  if (warp == 0 && on) {
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < GL_WARPS; i++) o += red[i * 32 + lane];
+    out[p.oa + h * E + e] = o;
+  }
+}
+
+__host__ __device__ inline int recur_blocks(const RecurP& p) {
+  return p.kind == MIX_GLA ? p.H * ((p.E + GL_COLS - 1) / GL_COLS) : p.H;
+}
+
 template <typename KT, int RM, bool FAST>
 __global__ void __launch_bounds__(MX_THREADS, 2) mixers_decode_kernel(const __grid_constant__ DecodeArgs a) {
   extern __shared__ __align__(16) float sm[];
@@ -563,11 +634,13 @@ __global__ void __launch_bounds__(MX_THREADS, 2) mixers_decode_kernel(const __gr
   int b = blockIdx.x;
   // recurrent heads first: they move the most bytes per block
   for (int i = 0; i < a.n_rec; i++) {
-    if (b < a.rec[i].H) {
-      recur_decode_head(a.rec[i], b, a.proj, a.out, pos, sm);
-          return;
+    const int n = recur_blocks(a.rec[i]);
+    if (b < n) {
+      if (a.rec[i].kind == MIX_GLA) gla_decode_unit(a.rec[i], b, a.proj, a.out, pos, sm);
+      else recur_decode_head(a.rec[i], b, a.proj, a.out, pos, sm);
+      return;
     }
-    b -= a.rec[i].H;
+    b -= n;
   }
   if (FAST) attn_decode_unit16<RM>(a.at, b, a.proj, a.out, pos, sm);
   else attn_decode_unit<KT, RM>(a.at, b, a.proj, a.out, pos, sm);
@@ -747,20 +820,23 @@ __global__ void conv_ring_kernel(const __grid_constant__ ConvP p, const float* _
 }
 
 // The recurrence of a pass: LPC lanes share one state column, RPL rows each, in registers for all
-// rows of the pass.  Rows of k, q and v of SC_T tokens at a time through shared memory.
+// rows of the pass.  Rows of k, q and v (gla: and of the decays) of SC_T tokens at a time through shared
+// memory.  `gates`: (step size, rate) per head, or the rates per key channel of gla.
 constexpr int SC_T = 16, SC_WARPS = 4;
 
-template <bool DELTA, int LPC, int RPL>
+template <int KIND, int LPC, int RPL>
 __global__ void __launch_bounds__(SC_WARPS * 32) recur_scan_kernel(const __grid_constant__ RecurP p,
-                                                                   const float* __restrict__ conv,
-                                                                   const float2* __restrict__ gates,
+                                                                   const float* __restrict__ conv, long long ld,
+                                                                   const void* __restrict__ gates,
                                                                    float* __restrict__ o, int rows, int pos0) {
+  constexpr bool DELTA = KIND == MIX_DELTA, GLA = KIND == MIX_GLA;
   constexpr int CPW = 32 / LPC, CPB = CPW * SC_WARPS, DR = LPC * RPL;
   extern __shared__ __align__(16) float sm[];
   float* ks = sm;                  // [SC_T][DR]
   float* qs = ks + SC_T * DR;      // [SC_T][DR]
   float* vs = qs + SC_T * DR;      // [SC_T][CPB]
   float2* gs = (float2*)(vs + SC_T * CPB);
+  float* as = (float*)(gs + SC_T);  // gla: [SC_T][DR]
   pdl_wait();
   pdl_launch_dependents();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -779,21 +855,22 @@ __global__ void __launch_bounds__(SC_WARPS * 32) recur_scan_kernel(const __grid_
     __syncthreads();
     for (int i = tid; i < n * DR; i += SC_WARPS * 32) {
       const int t = i / DR, d = i - t * DR;
-      const float* src = conv + (size_t)(tb + t) * p.cv.C;
+      const float* src = conv + (size_t)(tb + t) * ld;
       ks[i] = d < D ? src[p.ck + kg * D + d] : 0.f;
-      qs[i] = d < D ? src[p.cq + kg * D + d] : 0.f;
+      qs[i] = d < D ? (GLA ? src[p.cq + kg * D + d] * rsqrtf((float)D) : src[p.cq + kg * D + d]) : 0.f;
+      if (GLA) as[i] = d < D ? decay_of(((const float*)gates)[((size_t)(tb + t) * p.H + h) * D + d]) : 0.f;
     }
     for (int i = tid; i < n * CPB; i += SC_WARPS * 32) {
       const int t = i / CPB, c = i - t * CPB;
-      vs[i] = c0 + c < E ? conv[(size_t)(tb + t) * p.cv.C + p.cvv + h * E + c0 + c] : 0.f;
+      vs[i] = c0 + c < E ? conv[(size_t)(tb + t) * ld + p.cvv + h * E + c0 + c] : 0.f;
     }
-    if (tid < n) {
-      const float2 gt = gates[(size_t)(tb + tid) * p.H + h];
+    if (!GLA && tid < n) {
+      const float2 gt = ((const float2*)gates)[(size_t)(tb + tid) * p.H + h];
       gs[tid] = make_float2(gt.x, decay_of(gt.y));
     }
     __syncthreads();
     for (int t = 0; t < n; t++) {
-      const float2 gt = gs[t];
+      const float2 gt = GLA ? make_float2(0.f, 0.f) : gs[t];
       const float v = vs[t * CPB + cl];
       const float4* k4 = (const float4*)(ks + t * DR) + lr;
       const float4* q4 = (const float4*)(qs + t * DR) + lr;
@@ -815,6 +892,14 @@ __global__ void __launch_bounds__(SC_WARPS * 32) recur_scan_kernel(const __grid_
 #pragma unroll
         for (int w = LPC / 2; w > 0; w >>= 1) d0 += __shfl_xor_sync(0xffffffffu, d0, w);
         u = gt.x * (v - d0);
+      } else if (GLA) {
+        u = v;
+        const float4* a4 = (const float4*)(as + t * DR) + lr;
+#pragma unroll
+        for (int i = 0; i < RPL; i += 4) {
+          const float4 x = a4[(i >> 2) * LPC];
+          s[i] *= x.x; s[i + 1] *= x.y; s[i + 2] *= x.z; s[i + 3] *= x.w;
+        }
       } else {
         u = gt.x * v;
 #pragma unroll
@@ -857,7 +942,7 @@ __device__ __forceinline__ float sq4(float4 v, float s) {
   return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s))));
 }
 
-// delta rule: per-head norm, gate.  One warp per (row, head).
+// delta rule and gla: per-head norm, gate.  One warp per (row, head).
 template <typename OT>
 __global__ void __launch_bounds__(256) delta_finish_kernel(const __grid_constant__ RecurP p, const float* __restrict__ o,
                                                            const float* __restrict__ proj, long long ld,
@@ -944,7 +1029,10 @@ size_t attn_smem(const AttnP& p, int rm) {
   const int fast = p.Dp <= 128 && p.Ep <= 128 ? 8 * rm * p.Ep + 128 : 0;
   return (size_t)(rm * (2 * p.Dp + p.Ep + MX_TK) + 32 + 40 + 2 * p.Dp + p.Ep + fast) * sizeof(float);
 }
-size_t recur_smem(const RecurP& p) { return (size_t)(4 * p.D + 3 * p.E + 2 * MX_THREADS + 40) * sizeof(float); }
+size_t recur_smem(const RecurP& p) {
+  if (p.kind == MIX_GLA) return (size_t)(3 * p.D + MX_THREADS) * sizeof(float);
+  return (size_t)(4 * p.D + 3 * p.E + 2 * MX_THREADS + 40) * sizeof(float);
+}
 int rm_of(int hpb) { return hpb <= 1 ? 1 : (hpb <= 2 ? 2 : (hpb <= 4 ? 4 : 8)); }
 
 template <typename KT, int RM, bool FAST>
@@ -966,24 +1054,26 @@ int attn_rows_t(const AttnP& p, const void* q, const float* proj, long long ld, 
   TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, attn_rows_kernel<KT, RM>, p, (const KT*)q, proj, ld, (KT*)act, lda, pos0));
   return TLB_OK;
 }
-template <bool DELTA, int LPC, int RPL>
-int scan_t(const RecurP& p, const float* conv, const float2* gates, float* o, int rows, int pos0, cudaStream_t s) {
+template <int KIND, int LPC, int RPL>
+int scan_t(const RecurP& p, const float* conv, long long ld, const void* gates, float* o, int rows, int pos0,
+           cudaStream_t s) {
   constexpr int CPB = 32 / LPC * SC_WARPS, DR = LPC * RPL;
-  const size_t smem = (size_t)(2 * SC_T * DR + SC_T * CPB + 2 * SC_T) * sizeof(float);
+  const size_t smem = (size_t)((KIND == MIX_GLA ? 3 : 2) * SC_T * DR + SC_T * CPB + 2 * SC_T) * sizeof(float);
   static std::atomic<unsigned long long> done{0};
-  const int rc = ensure_dynamic_smem(recur_scan_kernel<DELTA, LPC, RPL>, 200 * 1024, done);
+  const int rc = ensure_dynamic_smem(recur_scan_kernel<KIND, LPC, RPL>, 200 * 1024, done);
   if (rc) return rc;
   LaunchCfg lc(dim3((p.E + CPB - 1) / CPB, p.H), dim3(SC_WARPS * 32), smem, s, pdl_enabled());
-  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, recur_scan_kernel<DELTA, LPC, RPL>, p, conv, gates, o, rows, pos0));
+  TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, recur_scan_kernel<KIND, LPC, RPL>, p, conv, ld, gates, o, rows, pos0));
   return TLB_OK;
 }
-template <bool DELTA>
-int scan_d(const RecurP& p, const float* conv, const float2* gates, float* o, int rows, int pos0, cudaStream_t s) {
-  if (p.D <= 32) return scan_t<DELTA, 8, 4>(p, conv, gates, o, rows, pos0, s);
-  if (p.D <= 64) return scan_t<DELTA, 8, 8>(p, conv, gates, o, rows, pos0, s);
-  if (p.D <= 128) return scan_t<DELTA, 8, 16>(p, conv, gates, o, rows, pos0, s);
-  if (p.D <= 256) return scan_t<DELTA, 8, 32>(p, conv, gates, o, rows, pos0, s);
-  if (p.D <= 1024) return scan_t<DELTA, 32, 32>(p, conv, gates, o, rows, pos0, s);
+template <int KIND>
+int scan_d(const RecurP& p, const float* conv, long long ld, const void* gates, float* o, int rows, int pos0,
+           cudaStream_t s) {
+  if (p.D <= 32) return scan_t<KIND, 8, 4>(p, conv, ld, gates, o, rows, pos0, s);
+  if (p.D <= 64) return scan_t<KIND, 8, 8>(p, conv, ld, gates, o, rows, pos0, s);
+  if (p.D <= 128) return scan_t<KIND, 8, 16>(p, conv, ld, gates, o, rows, pos0, s);
+  if (p.D <= 256) return scan_t<KIND, 8, 32>(p, conv, ld, gates, o, rows, pos0, s);
+  if (p.D <= 1024) return scan_t<KIND, 32, 32>(p, conv, ld, gates, o, rows, pos0, s);
   return set_error(TLB_ERR_UNSUPPORTED, "recurrent mixer: state width above 1024");
 }
 
@@ -1006,7 +1096,7 @@ int mixers_decode_launch(const AttnP* attn, const RecurP* rec, int n_rec, const 
   int blocks = a.n_attn;
   for (int i = 0; i < n_rec; i++) {
     a.rec[i] = rec[i];
-    blocks += rec[i].H;
+    blocks += recur_blocks(rec[i]);
     const size_t n = recur_smem(rec[i]);
     smem = n > smem ? n : smem;
   }
@@ -1060,16 +1150,17 @@ int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int
   return TLB_OK;
 }
 
-int recur_rows_scan_launch(const RecurP& p, const float* conv, const float2* gates, float* o, int rows, int pos0,
-                           cudaStream_t s) {
-  return p.kind == MIX_DELTA ? scan_d<true>(p, conv, gates, o, rows, pos0, s)
-                             : scan_d<false>(p, conv, gates, o, rows, pos0, s);
+int recur_rows_scan_launch(const RecurP& p, const float* conv, long long ld, const void* gates, float* o, int rows,
+                           int pos0, cudaStream_t s) {
+  if (p.kind == MIX_GLA) return scan_d<MIX_GLA>(p, conv, ld, gates, o, rows, pos0, s);
+  return p.kind == MIX_DELTA ? scan_d<MIX_DELTA>(p, conv, ld, gates, o, rows, pos0, s)
+                             : scan_d<MIX_SSD>(p, conv, ld, gates, o, rows, pos0, s);
 }
 
 int recur_rows_finish_launch(const RecurP& p, const float* o, const void* conv, bool conv_bf16, const float* proj,
                              long long ld, void* act, long long lda, int norm_groups, int rows, bool bf16, cudaStream_t s) {
   using B = __nv_bfloat16;
-  if (p.kind == MIX_DELTA) {
+  if (p.kind != MIX_SSD) {
     LaunchCfg lc(dim3(rows), dim3(256), 0, s, pdl_enabled());
     if (bf16) TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, delta_finish_kernel<B>, p, o, proj, ld, (B*)act, lda));
     else TLB_CUDA(cudaLaunchKernelEx(&lc.cfg, delta_finish_kernel<float>, p, o, proj, ld, (float*)act, lda));

@@ -11,10 +11,15 @@
 //               per-head RMS norm, silu output gate
 //   ssd         Mamba-2: one convolution over x | B | C, scalar-decay recurrence, skip, silu gate
 //               (the grouped norm behind it belongs to the output projection's input)
+//   latent      attention over a low-rank latent that all heads share: queries through a latent of their
+//               own, keys and values expanded per head from the kept latent beside one rotated key part,
+//               optional sliding window and sigmoid output gate (attn_latent.cu)
+//   gla         gated linear attention: one decay per key channel, per-head RMS norm, silu output gate
+//               (the norm and the gate belong to the output projection's input; prompts: recur_gla.cu)
 //
 // What a sequence carries is addressed by absolute position, so nothing is cleared between
-// sequences: keys and values live in kept slots plus a ring, the convolutions' inputs in a ring of
-// `taps` rows, and a recurrent state is read as zero at position 0.
+// sequences: keys and values live in kept slots plus a ring, latents in a ring, the convolutions' inputs in
+// a ring of `taps` rows, and a recurrent state is read as zero at position 0.
 #pragma once
 
 #include <cuda_bf16.h>
@@ -23,11 +28,12 @@
 
 namespace tlb {
 
-enum : int { MIX_ATTN = 1, MIX_DELTA = 2, MIX_SSD = 3 };
+enum : int { MIX_ATTN = 1, MIX_DELTA = 2, MIX_SSD = 3, MIX_LATENT = 4, MIX_GLA = 5 };
 
 struct AttnP {
   int H, G, D, E;              // query heads, key/value heads, query/key width, value width
   int Dp, Ep;                  // cache row lengths (widths rounded up to 8)
+  int Vs;                      // stride of value rows (a latent's value is a part of its key row)
   int window, keep, pairs;     // pairs = rotated dimensions / 2
   int oq, ok, ov, og;          // parts of the projected row
   int oa;                      // part of the finished row
@@ -46,6 +52,23 @@ __host__ __device__ inline size_t attn_part_floats(const AttnP& p) {
   return ((size_t)p.splits * p.hpb * (p.Ep + 2) + 3) & ~(size_t)3;
 }
 
+struct LatentP {
+  int H, D, R, E, Q, C;        // heads; unrotated, rotated and value width; query and key/value rank
+  int Dp, Rp, Ep, Qp, Cp;      // the same rounded up to 8
+  int window, ring;            // visible positions; kept rows
+  int oq, oc, og, oa;          // query latent, latent (rotated part behind it at oc + Cp), gate (-1: none),
+                               // part of the finished row
+  bool owner;                  // keeps rows of its own
+  float scale, eps, out_scale;
+  const float *qn, *cn;        // norms of the two latents
+  const float2* inv_freq;      // [R / 2]
+  const void *uq, *ukv;        // [H * (Dp + Rp)][Qp]; [H * Dp + H * Ep][Cp]
+  void* rows;                  // [ring][Cp + Rp]: latent | rotated key part
+  int splits;                  // most key ranges of a position
+  __host__ __device__ int row() const { return Cp + Rp; }
+  __host__ __device__ int qw() const { return Dp + Rp; }    // of a query head
+};
+
 struct ConvP {
   const float *w, *b;          // [C][taps], [C] or NULL
   float* ring;                 // [taps][C]: the row of position p sits at p % taps
@@ -53,15 +76,18 @@ struct ConvP {
 };
 
 struct RecurP {
-  int kind;                    // MIX_DELTA / MIX_SSD
+  int kind;                    // MIX_DELTA / MIX_SSD / MIX_GLA
   int H, G, D, E;              // heads, key groups, key (state) width, value width
   ConvP cv;
   int cq, ck, cvv;             // channel of the first query (C), key (B) and value (x)
-  int og, ob, oa_;             // gate (z), b (dt) and a parts of the projected row
+  int og, ob, oa_;             // gate (z), b (dt, decay input) and a parts of the projected row
   int oa;                      // part of the finished row
   float eps, out_scale;
   const float *A_log, *dt_bias, *Dskip, *norm;
   float* S;                    // [H][D][E]
+  int rank;                    // gla: decay input; cq, ck, cvv are parts of the projected row
+  float tau;
+  const float *a_up, *a_bias;  // [rank][H * D], [H * D]
 };
 
 #ifdef __CUDACC__
@@ -74,6 +100,7 @@ __device__ __forceinline__ float glu_clipped(float gate, float up, float limit) 
   const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
   return g * sigmoid_f(1.702f * g) * (u + 1.0f);
 }
+__device__ __forceinline__ float relu2(float z) { const float r = fmaxf(z, 0.f); return r * r; }
 
 // The same value in every thread of the block; sm holds 33 floats.  Barriers inside.
 __device__ __forceinline__ float block_sum(float v, float* sm) {
@@ -164,7 +191,7 @@ __device__ void attn_range(const AttnP& p, const float* qs, int g, const Visible
   constexpr int CE = Vec16<KT>::N;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const KT* K = (const KT*)p.K + (size_t)g * p.cap * p.Dp;
-  const KT* V = (const KT*)p.V + (size_t)g * p.cap * p.Ep;
+  const KT* V = (const KT*)p.V + (size_t)g * p.cap * p.Vs;
   float* corr = ml + 2 * RM;
   if (tid < RM) { ml[tid] = -3.0e38f; ml[RM + tid] = 0.f; }
   const int nc2 = p.Ep / 2, ngrp = MX_THREADS / nc2 < 1 ? 1 : MX_THREADS / nc2;
@@ -229,7 +256,7 @@ __device__ void attn_range(const AttnP& p, const float* qs, int g, const Visible
 #pragma unroll 4
       for (int k = grp; k < n; k += ngrp) {
         float a, b;
-        load2(V + (size_t)kv_slot(p, visible_pos(vis, tb + k)) * p.Ep + col, a, b);
+        load2(V + (size_t)kv_slot(p, visible_pos(vis, tb + k)) * p.Vs + col, a, b);
 #pragma unroll
         for (int r = 0; r < RM; r++) {
           const float w = sc[r * MX_TK + k];
@@ -279,6 +306,9 @@ __device__ __forceinline__ float2 recur_gates(const RecurP& p, const float* row,
   return make_float2(dt, expf(p.A_log[h]) * dt);
 }
 
+// -log of a gla decay: z is the sum behind the decay's projections
+__device__ __forceinline__ float gla_rate(float z, float tau) { return softplus_f(-z) / tau; }
+
 #endif  // __CUDACC__
 
 // launchers (mixers.cu, rows.cu)
@@ -290,6 +320,20 @@ int attn_rows_launch(const AttnP& p, const void* q, const float* proj, long long
                      int pos0, bool bf16, cudaStream_t s);
 // the same on the tensor pipe (attn_window.cu): bf16, widths up to 128
 bool attn_window_eligible(const AttnP& p);
+// the kernel behind it: where the rows of queries, keys (a part of their own and a shared part behind it)
+// and values lie; strides in elements, widths multiples of 8
+struct AttnTiles {
+  const void *q, *k, *k2, *v;
+  long long q_row, q_head, k_row, k_head, k2_row, v_row, v_head;
+  int kw, k2w, vw;             // widths of the key parts and of a value row; a query has kw + k2w
+  int H, R, E;                 // heads, heads on one key head, value width
+  int window, keep, ring;
+  float scale, out_scale;
+  const float* gate;           // [row][gate_row], head h at h * E; NULL: none
+  long long gate_row;
+};
+bool attn_tiles_eligible(int qk_width, int v_width);
+int attn_tiles_launch(const AttnTiles& t, void* out, long long ldo, int rows, int pos0, cudaStream_t s);
 int attn_window_launch(const AttnP& p, const void* q, const float* proj, long long ld, void* act, long long lda,
                        int rows, int pos0, cudaStream_t s);
 // Convolutions, step sizes and rates of a pass, in one of two forms: f32 with the delta rule's unit
@@ -297,8 +341,9 @@ int attn_window_launch(const AttnP& p, const void* q, const float* proj, long lo
 // with the factors that make queries and keys unit vectors apart ([rows][G] query, key), for the chunks.
 int recur_rows_conv_launch(const RecurP& p, const float* proj, long long ld, int rows, int pos0, void* conv,
                            float2* gates, float2* norms, bool chunked, cudaStream_t s);
-int recur_rows_scan_launch(const RecurP& p, const float* conv, const float2* gates, float* o, int rows, int pos0,
-                           cudaStream_t s);
+// gla: conv is the projected rows (stride ld), gates the rates [rows][H * D]
+int recur_rows_scan_launch(const RecurP& p, const float* conv, long long ld, const void* gates, float* o, int rows,
+                           int pos0, cudaStream_t s);
 int recur_rows_finish_launch(const RecurP& p, const float* o, const void* conv, bool conv_bf16, const float* proj,
                              long long ld, void* act, long long lda, int norm_groups, int rows, bool bf16, cudaStream_t s);
 // the recurrence in chunks on the tensor pipe (recur_chunk.cu)
@@ -306,12 +351,42 @@ bool recur_chunk_eligible(const RecurP& p);
 size_t recur_chunk_scratch_bytes(const RecurP& p, int rows);
 int recur_chunk_launch(const RecurP& p, const void* conv, const float2* gates, const float2* norms, void* scratch,
                        float* o, int rows, int pos0, cudaStream_t s);
-int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, long long ldo, int n, float eps, int rows,
-                    bool bf16, cudaStream_t s);
+// gated linear attention of a pass (recur_gla.cu): rates of every row and key channel, then the recurrence
+// token by token or in chunks on the tensor pipe (bf16)
+int gla_rates_launch(const RecurP& p, const float* proj, long long ld, float* rates, int rows, cudaStream_t s);
+bool gla_chunk_eligible(const RecurP& p);
+size_t gla_chunk_scratch_bytes(const RecurP& p, int rows);
+int gla_chunk_launch(const RecurP& p, const float* proj, long long ld, const float* rates, void* scratch, float* o,
+                     int rows, int pos0, cudaStream_t s);
+
+// latent attention (attn_latent.cu).  `rows` positions from *d_pos (one token) or from pos0:
+//   prep     (prompt pass) normed query latents, kept rows
+//   absorb   queries against the latent, rotated; with d_pos the token's kept row
+//   attend   weighted latents of key ranges, with their maxima and sums
+//   fold     ranges merged, values, gate
+// or, for many rows in bf16: q_rows (rotated queries) and attn_tiles on expanded keys and values
+size_t latent_part_floats(const LatentP& p, int rows, int splits);
+int latent_splits(const LatentP& p, int rows);
+int latent_prep_launch(const LatentP& p, const float* proj, long long ld, int rows, int pos0, void* qlat, bool bf16,
+                       cudaStream_t s);
+int latent_absorb_launch(const LatentP& p, const float* q, long long ldq, const float* proj, void* qa, int rows,
+                         const unsigned* d_pos, int pos0, bool bf16, cudaStream_t s);
+int latent_attend_launch(const LatentP& p, const void* qa, float* part, int rows, int splits, const unsigned* d_pos,
+                         int pos0, bool bf16, cudaStream_t s);
+int latent_fold_launch(const LatentP& p, const float* part, int splits, const float* proj, long long ld, void* act,
+                       long long lda, int rows, const unsigned* d_pos, int pos0, bool bf16, bool act_bf16, cudaStream_t s);
+int latent_q_rows_launch(const LatentP& p, const float* q, long long ldq, void* out, int rows, int pos0, cudaStream_t s);
+
+int rms_rows_launch(const float* x, long long ldx, const float* w, void* out, long long ldo, int n, float eps,
+                    float scale, int rows, bool bf16, cudaStream_t s);
+// x += norm(y) (y NULL: x as it is), and the result as the next product's operand
+int residual_rows_launch(float* x, const float* y, const float* w, void* out, long long ldo, int n, float eps, int rows,
+                         bool bf16, cudaStream_t s);
 int embed_scaled_launch(const void* embed, const int* ids, float* x, int width, long long ld, float scale, int rows,
                         bool bf16, cudaStream_t s);
 int gather_rows_launch(const float* x, const int* idx, float* out, int width, int rows, cudaStream_t s);
 int glu_rows_launch(const float* gu, float* out, int ff, float limit, int rows, cudaStream_t s);
+int relu2_rows_launch(const float* u, float* out, int ff, int rows, cudaStream_t s);
 
 // one-row matrix product with its neighbours fused (gemv_rows.cu)
 struct RowGemv {
@@ -324,8 +399,12 @@ struct RowGemv {
   const float* nw;
   int n_off, n_len, n_groups;
   float eps, nscale;
+  const float* gate;         // [n_len] the normed part times silu(gate) (NULL: none)
+  // a residual in front of it all: the row becomes res + norm(x) * rn, block 0 leaves it in xout
+  const float *res, *rn;
+  float* xout;
   float* y;
-  int epi;                   // 0 y = , 1 y += , 2 y[j] = glu(row 2j, row 2j + 1)
+  int epi;                   // 0 y = , 1 y += , 2 y[j] = glu(row 2j, row 2j + 1), 3 y = relu2
   float limit;
 };
 int row_gemv_launch(DeviceCtx* c, const RowGemv& p, bool bf16, cudaStream_t s);

@@ -12,6 +12,7 @@ from .safetensors import SafeTensors
 ARCHITECTURES = {
     "Qwen2ForCausalLM": "cpp_tensorlib_b200.decoder:Q4Decoder",
     "Zavilorn": "cpp_tensorlib_b200.zavilorn:Zavilorn",
+    "Daronex": "cpp_tensorlib_b200.daronex:Daronex",
 }
 DTYPES = ("bfloat16", "float32")
 

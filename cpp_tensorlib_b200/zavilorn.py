@@ -122,8 +122,8 @@ class RandomTensors:
     SafeTensors).  Matrices have standard deviation 1 / sqrt(columns), norms are near one, decay rates
     and step biases lie where the recurrences remember tens to hundreds of tokens."""
 
-    def __init__(self, config, seed=0, pool=1 << 24):
-        self.shapes = tensor_shapes(config)
+    def __init__(self, config, seed=0, pool=1 << 24, shapes=None):
+        self.shapes = shapes or tensor_shapes(config)
         self.rng = np.random.default_rng(seed)
         self.pool = self.rng.standard_normal(pool, dtype=np.float32)
 

@@ -283,45 +283,65 @@ int tlb_decoder_prefill_logits(void* dec, const int32_t* tokens, int64_t T, cons
  * of it is addressed by position, so tlb_decoder_set_pos(dec, 0) starts a new sequence; any other
  * move than to the current position is refused.
  *
+ * Latent attention keeps one row per position for all its heads (the normed latent and the rotated key
+ * part they share); a layer may read the rows of an earlier layer instead of keeping its own.
+ *
  * The projected row of a layer is the mixers' parts one after the other, every part padded to a
  * multiple of 8 rows (zero weight rows):
  *   attention   q [heads*dim] | k [kv_heads*dim] | v [kv_heads*vdim] | gate [heads*vdim]
  *   delta rule  q [kv_heads*dim] | k [kv_heads*dim] | v [heads*vdim] | gate [heads*vdim] | b [heads] | a [heads]
  *   ssd         z [heads*vdim] | x,B,C [heads*vdim + 2*kv_heads*dim] (one part) | dt [heads]
+ *   latent      query latent [q_rank] | latent [kv_rank] | rotated key part [rot_dims] (these two only
+ *               without kv_from) | gate [heads*vdim] (with gate)
+ *   gla         q [heads*dim] | k [heads*dim] | v [heads*vdim] | gate [heads*vdim] | decay input [rank]
  * Convolution weights cover the padded channels of q | k | v, or of x,B,C.  The row the output
  * projection reads is the mixers' heads, [heads*vdim] each, padded to multiples of 8. ---- */
 #define TLB_MIX_ATTN 1
 #define TLB_MIX_DELTA 2
 #define TLB_MIX_SSD 3
+#define TLB_MIX_LATENT 4
+#define TLB_MIX_GLA 5
 typedef struct {
   int32_t kind;
   int32_t heads, kv_heads;        /* ssd: kv_heads = groups */
   int32_t dim, vdim;              /* ssd: dim = state width */
-  int32_t window, keep_first;     /* attention */
-  int32_t rot_dims;
+  int32_t window, keep_first;     /* attention; latent: window 0 = everything before */
+  int32_t rot_dims;               /* of dim; latent: dimensions beside dim, all of them rotated */
   int32_t conv;                   /* taps, recurrent mixers */
   int32_t norm_groups;            /* ssd */
-  float rot_base, scale;          /* attention */
+  int32_t q_rank, kv_rank;        /* latent */
+  int32_t gate;                   /* latent: 1 = sigmoid output gate */
+  int32_t kv_from;                /* latent: layer whose kept rows it reads, -1 = its own */
+  int32_t rank;                   /* gla: width of the decay's input */
+  float rot_base, scale;          /* attention, latent */
   float out_scale;                /* factor of the mixer's result in the layer */
+  float tau;                      /* gla: decay = sigmoid(.)^(1/tau) */
 } tlb_mixer_cfg;
 typedef struct {
   int32_t n_mixers;
   int32_t ff;                     /* 0: no feed-forward */
+  int32_t act;                    /* 0: clipped gated unit, 1: square of relu */
   float limit;                    /* clipped gated unit */
   tlb_mixer_cfg mixer[2];
 } tlb_layer_cfg;
 typedef struct {
   int32_t width, vocab, n_layers, max_ctx, f32;
-  float eps, embed_scale;
+  int32_t post_norm;              /* 0: x += f(norm(x)), 1: x += norm(f(x)) */
+  float eps, embed_scale, logit_scale;
 } tlb_stack_cfg;
 int tlb_stack_create(const tlb_stack_cfg* cfg, const tlb_layer_cfg* layers, void** out);
 /* HOST matrices [rows, cols] in the model's type, copied to the device.  which: 0 input projection,
- * 1 output projection, 2 gate and up rows interleaved [2*ff, width], 3 down [width, ff], 4 embedding
- * [vocab, width] (also the output head; layer ignored). */
+ * 1 output projection, 2 gate and up rows interleaved [2*ff, width] (act 1: up [ff, width]), 3 down
+ * [width, ff], 4 embedding [vocab, width], 5 output head [vocab, width] (never set: the embedding); 4 and
+ * 5 ignore the layer.  Of latent mixer m: 16 + m queries from their latent, per head [dim padded to 8 |
+ * rot_dims padded to 8] rows by q_rank; 24 + m keys, per head [dim padded to 8], then values, per head
+ * [vdim padded to 8] rows, by kv_rank.  Rotated rows come in adjacent pairs. */
 int tlb_stack_set_matrix(void* dec, int64_t layer, int which, const void* w, int64_t rows, int64_t cols);
-/* HOST f32 vectors.  which: 0 norm in front of the mixers, 1 norm in front of the feed-forward,
+/* HOST f32 vectors.  which: 0 norm in front of the mixers, 1 norm in front of the feed-forward (post_norm: both behind),
  * 2 final norm (layer ignored); of mixer m: 10 + query norm 0, key norm 1, output norm 2,
- * convolution weights [channels, taps] 3, convolution bias 4, step bias 5, log decay rate 6, skip 7. */
+ * convolution weights [channels, taps] 3, convolution bias 4, step bias 5, log decay rate 6, skip 7, decay
+ * weights [rank, heads*dim] 8, decay bias [heads*dim] 9.  Latent: query latent's norm 10, latent's norm
+ * 11.  The output norm of gla has heads*vdim weights. */
 int tlb_stack_set_vector(void* dec, int64_t layer, int mixer, int which, const float* v, int64_t n);
 /* Bytes of sequence state (caches, rings, recurrent states) the decoder holds. */
 int64_t tlb_stack_state_bytes(void* dec);
