@@ -300,68 +300,108 @@ def zavilorn_config(size):
                 layers=[par, mam, mam, mam] * 2)
 
 
+def daronex_config(size):
+    """Layers of a real model's proportions at Zavilorn's sizes: latent attentions of the whole context (the
+    second on the first one's latent) and of a window, each followed by a gated linear attention."""
+    w, heads, q_rank, ff = dict(small=(2048, 16, 1024, 8192), medium=(4096, 32, 1536, 16384))[size]
+    lat = dict(heads=heads, dim=128, rot_dim=64, vdim=128, q_rank=q_rank, kv_rank=512, rot=dict(base=1e5, dims=64),
+               scale=192 ** -0.5)
+    mlp = dict(kind="dense", ff=ff)
+    gla = dict(type="gla", mlp=mlp, mixer=dict(heads=w // 256, dim=128, vdim=256, tau=16.0))
+    win = dict(type="latent_attention_2", mlp=mlp, mixer=dict(lat, mask=dict(size=2048)))
+    return dict(architecture="Daronex", vocab=65536, width=w, norm=dict(eps=1e-6), logit_scale=1.0, layers=[
+        dict(type="latent_attention", mlp=mlp, mixer=lat), gla, win, gla,
+        dict(type="latent_attention", mlp=mlp, mixer=dict(lat, kv_from=0)), gla, win, gla])
+
+
+def matrix_elements(shapes, tables):
+    """Elements of the matrices a token multiplies with; `tables` name the ones it does not."""
+    return sum(s[0] * s[1] for n, s in shapes.items() if len(s) == 2 and not n.endswith("conv") and n not in tables)
+
+
+def model_arms(name, size, T):
+    """(name, config, constructor of the loaded model, matrix elements of a token, sequence state read and
+    written per token behind T tokens) of a model and of its neighbours at equal size."""
+    from cpp_tensorlib_b200 import daronex, zavilorn
+    zc = zavilorn_config(size)
+    a = zc["layers"][0]["mixer"]["left"]
+
+    def load_zavilorn(max_ctx):
+        z = zavilorn.Zavilorn(zc, "bfloat16", max_ctx)
+        z.load(zavilorn.RandomTensors(zc, SEED))
+        return z
+    state = sum(2 * a["kv_heads"] * 128 * 2 * min(T, a["mask"]["size"] + 4) for L in zc["layers"] if L["type"] == "parallel")
+    state += sum(2 * 4 * (m["heads"] * m["vdim"] * m["state"] if L["type"] == "mamba2" else
+                          m["right"]["heads"] * 128 * 128) for L in zc["layers"] for m in [L["mixer"]])
+    zav = ("zavilorn", zc, load_zavilorn, matrix_elements(zavilorn.tensor_shapes(zc), ()), state)
+    qc = dict(hidden=zc["width"], layers=len(zc["layers"]), n_q=a["heads"], n_kv=a["kv_heads"], hd=128,
+              ff=zc["layers"][0]["mlp"]["ff"], vocab=zc["vocab"], eps=1e-6, rope_base=1e6)
+    if name == "zavilorn":
+        wb, kv, params = token_bytes(qc, T)
+        return [zav, ("q4", qc, lambda max_ctx: build_decoder(qc, max_ctx, 0, 1, 0), params, kv + wb - 2 * params)]
+    dc = daronex_config(size)
+
+    def load_daronex(max_ctx):
+        t = daronex.RandomTensors(dc, SEED)
+        return daronex.Daronex.from_folder(dc, t, "bfloat16", max_ctx)
+    state = 0
+    for L in dc["layers"]:
+        m = L["mixer"]
+        if L["type"] == "gla":
+            state += 2 * 4 * m["heads"] * m["dim"] * m["vdim"]
+        else:
+            state += 2 * (m["kv_rank"] + m["rot_dim"]) * min(T, m["mask"]["size"] if "mask" in m else T)
+    return [("daronex", dc, load_daronex, matrix_elements(daronex.tensor_shapes(dc), ("embed",)), state), zav]
+
+
 def run_model(args):
-    """Prefill and decode throughput of the layer-stack model (random weights, one GPU) beside the int4
-    decoder with the same width, heads, feed-forward, vocabulary and layer count.  One JSON line per size."""
+    """Prefill and decode throughput of a layer-stack model (random weights, one GPU) beside its closest
+    neighbour with the same width, heads, vocabulary and layer count.  One JSON line per size."""
     import torch
-    from cpp_tensorlib_b200.zavilorn import RandomTensors, Zavilorn
     torch.cuda.set_device(0)
     T, K, W = args.prefill or 4096, args.steps, max(3, args.warmup)
     peak, src = measured_peaks()
-    for size in args.size.split(","):
-        cfg = zavilorn_config(size)
-        a = cfg["layers"][0]["mixer"]["left"]
-        qcfg = dict(hidden=cfg["width"], layers=len(cfg["layers"]), n_q=a["heads"], n_kv=a["kv_heads"], hd=128,
-                    ff=cfg["layers"][0]["mlp"]["ff"], vocab=cfg["vocab"], eps=1e-6, rope_base=1e6)
-        ids = np_ids(cfg["vocab"], T)
-        line = dict(metric="prefill and decode tok/s", size=size, prompt=T, steps=K, warmup=W, n_gpus=1, data="synthetic",
-                    config=dict(zavilorn=cfg, q4=qcfg), peak_source=src)
 
-        def measure(d):
-            times = []
-            for _ in range(2 + max(1, args.repeats)):
-                d.set_pos(0)
-                torch.cuda.synchronize()
-                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-                e0.record()
-                d.prefill(ids)
-                e1.record()
-                torch.cuda.synchronize()
-                times.append(e0.elapsed_time(e1))
-            pre = statistics.median(times[2:])
-            d.capture()
-            d.run(W)
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    def measure(d, ids):
+        times = []
+        for _ in range(2 + max(1, args.repeats)):
+            d.set_pos(0)
             torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             e0.record()
-            d.run(K)
+            d.prefill(ids)
             e1.record()
             torch.cuda.synchronize()
-            dec = e0.elapsed_time(e1) / K
-            return dict(prefill_ms=pre, prefill_tok_s=T / pre * 1e3, decode_ms=dec, decode_tok_s=1e3 / dec,
-                        launches_per_token=d.launches_per_token())
+            times.append(e0.elapsed_time(e1))
+        pre = statistics.median(times[2:])
+        d.capture()
+        d.run(W)
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        d.run(K)
+        e1.record()
+        torch.cuda.synchronize()
+        dec = e0.elapsed_time(e1) / K
+        return dict(prefill_ms=pre, prefill_tok_s=T / pre * 1e3, decode_ms=dec, decode_tok_s=1e3 / dec,
+                    launches_per_token=d.launches_per_token())
 
+    for size in args.size.split(","):
+        line = dict(metric="prefill and decode tok/s", size=size, prompt=T, steps=K, warmup=W, n_gpus=1, data="synthetic",
+                    config={}, peak_source=src)
         with ClockSampler(0) as clk:
-            z = Zavilorn(cfg, "bfloat16", T + W + K + 8)
-            t = RandomTensors(cfg, SEED)
-            z.load(t)
-            mats = sum(s[0] * s[1] for n, s in t.shapes.items() if len(s) == 2 and not n.endswith("conv"))
-            r = measure(z)
-            z.close()
-            win = sum(2 * a["kv_heads"] * 128 * 2 * min(T, a["mask"]["size"] + 4) for L in cfg["layers"] if L["type"] == "parallel")
-            rec = sum(2 * 4 * (m["heads"] * m["vdim"] * m["state"] if L["type"] == "mamba2" else
-                               m["right"]["heads"] * 128 * 128) for L in cfg["layers"] for m in [L["mixer"]])
-            r.update(decode_bytes=2 * mats + win + rec, decode_frac_hbm=(2 * mats + win + rec) / r["decode_ms"] / 1e6 / peak,
-                     prefill_matrix_tflops=2 * (mats - cfg["vocab"] * cfg["width"]) * T / r["prefill_ms"] / 1e9)
-            line["zavilorn"] = r
-            if not args.no_q4:
-                q = build_decoder(qcfg, T + W + K + 8, 0, 1, 0)
-                r = measure(q)
-                q.close()
-                wb, kv, params = token_bytes(qcfg, T)
-                r.update(decode_bytes=wb + kv, decode_frac_hbm=(wb + kv) / r["decode_ms"] / 1e6 / peak,
-                         prefill_matrix_tflops=2 * (params - cfg["vocab"] * cfg["width"]) * T / r["prefill_ms"] / 1e9)
-                line["q4"] = r
+            for i, (name, cfg, load, mats, state) in enumerate(model_arms(args.model, size, T)):
+                line["config"][name] = cfg
+                if i and args.alone:
+                    continue
+                d = load(T + W + K + 8)
+                r = measure(d, np_ids(cfg["vocab"], T))
+                d.close()
+                width = cfg.get("width") or cfg["hidden"]
+                nbytes = 2 * mats + state
+                r.update(decode_bytes=nbytes, decode_frac_hbm=nbytes / r["decode_ms"] / 1e6 / peak,
+                         prefill_matrix_tflops=2 * (mats - cfg["vocab"] * width) * T / r["prefill_ms"] / 1e9)
+                line[name] = r
         line["clocks"] = clk.summary()
         print(json.dumps(line), flush=True)
 
@@ -381,11 +421,12 @@ def main():
     ap.add_argument("--prefill", type=int, default=0,
                     help="diagnostic: time the batched prompt pass over this many tokens and exit")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--model", default="q4", choices=["q4", "zavilorn"],
-                    help="zavilorn: prefill and decode of the layer-stack model beside the int4 decoder, then exit")
-    ap.add_argument("--size", default="small,medium", help="with --model zavilorn: sizes, with commas between them")
-    ap.add_argument("--repeats", type=int, default=5, help="with --model zavilorn: timed prompt passes")
-    ap.add_argument("--no-q4", action="store_true", help="with --model zavilorn: leave the int4 decoder out")
+    ap.add_argument("--model", default="q4", choices=["q4", "zavilorn", "daronex"],
+                    help="prefill and decode of a layer-stack model beside its closest neighbour (zavilorn: the int4 "
+                         "decoder, daronex: zavilorn), then exit")
+    ap.add_argument("--size", default="small,medium", help="with --model: sizes, with commas between them")
+    ap.add_argument("--repeats", type=int, default=5, help="with --model: timed prompt passes")
+    ap.add_argument("--alone", action="store_true", help="with --model: leave the neighbour out")
     args = ap.parse_args()
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
