@@ -161,7 +161,8 @@ __device__ __forceinline__ float2* stat_of(const LatentP& p, float* part, int sp
   return (float2*)(part + (size_t)rows * splits * p.H * p.Cp) + ((size_t)row * splits + split) * p.H;
 }
 
-// any widths, either type: block (range, RM heads, row)
+// any widths, either type: block (range, RM heads, row); 512 of the latent's columns at a time
+constexpr int LA_VALUES = 2 * MX_THREADS;
 template <typename KT, int RM>
 __global__ void __launch_bounds__(LA_THREADS) latent_attend_kernel(const __grid_constant__ LatentP p,
                                                                    const KT* __restrict__ qa, float* __restrict__ part,
@@ -174,20 +175,28 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attend_kernel(const __grid_
   pdl_launch_dependents();
   if ((int)blockIdx.x >= lr.active) return;
   AttnP a{};
-  a.Dp = p.row(); a.Ep = p.Cp; a.Vs = p.row(); a.cap = a.ring = p.ring; a.keep = 0; a.scale = p.scale;
-  a.K = a.V = p.rows;
+  a.Dp = p.row(); a.Vs = p.row(); a.cap = a.ring = p.ring; a.keep = 0; a.scale = p.scale;
+  a.K = p.rows;
   float* qs = sm;
   float* os = qs + RM * a.Dp;
-  float* sc = os + RM * a.Ep;
+  float* sc = os + RM * (p.Cp < LA_VALUES ? p.Cp : LA_VALUES);
   float* ml = sc + RM * MX_TK;
   for (int i = tid; i < RM * a.Dp; i += LA_THREADS)
     qs[i] = i < nh * a.Dp ? to_f(qa[((size_t)row * p.H + h0) * a.Dp + i]) : 0.f;
   Visible vis;
   vis.kept = 0; vis.lo = lr.lo; vis.n = lr.n;
   const int t0 = blockIdx.x * lr.chunk, t1 = t0 + lr.chunk < lr.n ? t0 + lr.chunk : lr.n;
-  attn_range<KT, RM>(a, qs, 0, vis, t0, t1, sc, os, ml);
   float* dst = part_of(p, part, splits, row, blockIdx.x) + (size_t)h0 * p.Cp;
-  for (int i = tid; i < nh * p.Cp; i += LA_THREADS) dst[i] = os[i];
+  for (int c0 = 0; c0 < p.Cp; c0 += LA_VALUES) {
+    a.V = (KT*)p.rows + c0;
+    a.Ep = p.Cp - c0 < LA_VALUES ? p.Cp - c0 : LA_VALUES;
+    __syncthreads();
+    attn_range<KT, RM>(a, qs, 0, vis, t0, t1, sc, os, ml);
+    for (int i = tid; i < nh * a.Ep; i += LA_THREADS) {
+      const int r = i / a.Ep;
+      dst[(size_t)r * p.Cp + c0 + i - r * a.Ep] = os[i];
+    }
+  }
   if (tid < nh) stat_of(p, part, splits, gridDim.z, row, blockIdx.x)[h0 + tid] = make_float2(ml[tid], ml[RM + tid]);
 }
 
@@ -227,13 +236,13 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attend_mma_kernel(const __g
   if ((int)blockIdx.x >= lr.active) { pdl_wait(); pdl_launch_dependents(); return; }
   const int t0 = blockIdx.x * lr.chunk, t1 = t0 + lr.chunk < lr.n ? t0 + lr.chunk : lr.n;
   const int ntile = (t1 - t0 + LM_KEYS - 1) / LM_KEYS;
-  auto fetch = [&](int tile, int buf) {
-    for (int i = tid; i < LM_KEYS * ch; i += LA_THREADS) {
-      const int r = i / ch, c = i - r * ch, t = t0 + tile * LM_KEYS + r;
-      const bool on = t < t1;
-      rc_cp16(ks + (buf * LM_KEYS + r) * ld + c * 8,
-              (const B*)p.rows + (size_t)latent_slot(p, lr.lo + (on ? t : t0)) * rw + c * 8, on);
-    }
+  auto fetch = [&](int tile, int buf) {   // four threads a row
+    const int r = tid >> 2, t = t0 + tile * LM_KEYS + r;
+    const bool on = t < t1;
+    const B* src = (const B*)p.rows + (size_t)latent_slot(p, lr.lo + (on ? t : t0)) * rw;
+    B* dst = ks + (buf * LM_KEYS + r) * ld;
+#pragma unroll 6
+    for (int c = tid & 3; c < ch; c += 4) rc_cp16(dst + c * 8, src + c * 8, on);
   };
   // columns that a product reads behind the row's own
   for (int i = tid; i < (16 + 2 * LM_KEYS) * (ld - rw) / 8; i += LA_THREADS) {
@@ -421,7 +430,10 @@ __global__ void __launch_bounds__(LA_THREADS) latent_fold_kernel(const __grid_co
     float f[CE];
     widen16(x, f, (const KT*)nullptr);
 #pragma unroll
-    for (int e = 0; e < CE; e++) s = fmaf(f[e], c[k * CE + e], s);
+    for (int e = 0; e < CE; e += 4) {
+      const float4 v = *(const float4*)(c + k * CE + e);
+      s = fmaf(f[e], v.x, fmaf(f[e + 1], v.y, fmaf(f[e + 2], v.z, fmaf(f[e + 3], v.w, s))));
+    }
   };
 #pragma unroll
   for (int j = 0; j < 2; j++) {
@@ -476,7 +488,8 @@ int attend_mma(const LatentP& p, const void* qa, float* part, int rows, int spli
 template <typename KT, int RM>
 int attend_any(const LatentP& p, const void* qa, float* part, int rows, int splits, const unsigned* d_pos, int pos0,
                cudaStream_t s) {
-  const size_t smem = (size_t)(RM * (p.row() + p.Cp + MX_TK) + 3 * RM + 32) * sizeof(float);
+  const int values = p.Cp < LA_VALUES ? p.Cp : LA_VALUES;
+  const size_t smem = (size_t)(RM * (p.row() + values + MX_TK) + 3 * RM + 32) * sizeof(float);
   static std::atomic<unsigned long long> done{0};
   const int rc = ensure_dynamic_smem(latent_attend_kernel<KT, RM>, 200 * 1024, done);
   if (rc) return rc;

@@ -3,7 +3,7 @@
 // The rates -log a_t of every row come first (gla_rates), f32 throughout.  f32 models then run the
 // recurrence token by token (recur_scan_kernel of mixers.cu).  bf16 models run it in chunks of 64 tokens on
 // the tensor pipe, with b_t the running sum of rates inside a chunk:
-//   gla_state  (chunk, head, 64 value columns)   U = sum_s exp(b_s - b_L) k_s v_s^T, and exp(-b_L)
+//   gla_state  (chunk, head, value columns)      U = sum_s exp(b_s - b_L) k_s v_s^T, and exp(-b_L)
 //   gla_carry  (state elements)                  S <- diag(exp(-b_L)) S + U down the chunks, each chunk's U
 //                                                replaced by the state in front of it
 //   gla_out    (chunk, head)                     o_t = (exp(-b_t) q_t) S + sum_{s <= t} A_ts v_s,
@@ -18,7 +18,7 @@ namespace tlb {
 
 namespace {
 
-constexpr int GC_L = 64, GC_E = 64, GC_THREADS = 256, GC_ELD = GC_E + 8;
+constexpr int GC_L = 64, GC_E = 64, GC_THREADS = 256, GC_ELD = GC_E + 8;   // GC_E: value columns of gla_out
 constexpr float GC_MOST = 60.f;   // largest b_L of the factored form
 
 // ---- rates ---------------------------------------------------------------------------------------
@@ -70,30 +70,38 @@ __device__ __forceinline__ void put_planes(__nv_bfloat16* at, size_t plane, floa
   at[0] = hi;
   at[plane] = __float2bfloat16_rn(v - __bfloat162float(hi));
 }
-// 64 rows x 64 columns of f32 rows as bf16; columns from c on beyond E and rows from n on are zero
-__device__ __forceinline__ void load_values(__nv_bfloat16* vs, const float* src, long long ld, int n, int cols) {
-  for (int i = threadIdx.x; i < GC_L * GC_E / 2; i += GC_THREADS) {
-    const int t = i / (GC_E / 2), c = (i - t * (GC_E / 2)) * 2;
-    const float* at = src + (size_t)t * ld + c;
-    const float a = t < n && c < cols ? at[0] : 0.f, b = t < n && c + 1 < cols ? at[1] : 0.f;
-    *(__nv_bfloat162*)(vs + t * GC_ELD + c) = __floats2bfloat162_rn(a, b);
+// four adjacent elements of a row of which `left` are there; vec: rows start on 16 bytes
+__device__ __forceinline__ float4 load4(const float* at, int left, bool vec) {
+  if (vec && left >= 4) return *(const float4*)at;
+  return make_float4(left > 0 ? at[0] : 0.f, left > 1 ? at[1] : 0.f, left > 2 ? at[2] : 0.f, left > 3 ? at[3] : 0.f);
+}
+// 64 rows x W columns of f32 rows as bf16; columns from `cols` on and rows from n on are zero
+template <int W>
+__device__ __forceinline__ void load_values(__nv_bfloat16* vs, const float* src, long long ld, int n, int cols, bool vec) {
+#pragma unroll 4
+  for (int i = threadIdx.x; i < GC_L * W / 4; i += GC_THREADS) {
+    const int t = i / (W / 4), c = (i - t * (W / 4)) * 4;
+    const float4 v = load4(src + (size_t)t * ld + c, t < n ? cols - c : 0, vec);
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *(uint2*)(vs + t * (W + 8) + c) = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
   }
 }
 
 // ---- what a chunk adds to the state -----------------------------------------------------------------
+template <int DP> constexpr int GS_E = DP <= 128 ? 128 : 64;   // value columns of a block
 template <int DP>
 __global__ void __launch_bounds__(GC_THREADS) gla_state_kernel(const __grid_constant__ RecurP p,
                                                                const float* __restrict__ proj, long long ld,
                                                                const float* __restrict__ rates, float* __restrict__ U,
                                                                float* __restrict__ decay, int rows) {
   constexpr int LD = DP + 8, NG = GC_THREADS / DP, TG = GC_L / NG, MT = DP >= 128 ? DP / 128 : 1;
-  constexpr int NT = DP >= 128 ? 4 : 2;        // pairs of column tiles of a warp
+  constexpr int SE = GS_E<DP>, SLD = SE + 8, NT = (DP >= 128 ? SE : SE / 2) / 16;   // pairs of column tiles of a warp
   extern __shared__ __align__(16) unsigned char smem[];
   __nv_bfloat16* ks = (__nv_bfloat16*)smem;    // [2 planes][64][LD]
-  __nv_bfloat16* vs = ks + 2 * GC_L * LD;      // [64][GC_ELD]
-  float* gsum = (float*)(vs + GC_L * GC_ELD);  // [NG][DP]
+  __nv_bfloat16* vs = ks + 2 * GC_L * LD;      // [64][SLD]
+  float* gsum = (float*)(vs + GC_L * SLD);     // [NG][DP]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, D = p.D, E = p.E;
-  const int e0 = blockIdx.x * GC_E, h = blockIdx.y, ch = blockIdx.z, t0 = ch * GC_L;
+  const int e0 = blockIdx.x * SE, h = blockIdx.y, ch = blockIdx.z, t0 = ch * GC_L;
   const int n = rows - t0 < GC_L ? rows - t0 : GC_L, d = tid % DP, grp = tid / DP, tg = grp * TG, HD = p.H * D;
   pdl_wait();
   pdl_launch_dependents();
@@ -102,7 +110,7 @@ __global__ void __launch_bounds__(GC_THREADS) gla_state_kernel(const __grid_cons
 #pragma unroll
   for (int i = 0; i < TG; i++) kv[i] = d < D && tg + i < n ? kr[(size_t)i * ld] : 0.f;
   gsum[grp * DP + d] = load_rates<TG>(rates + (size_t)(t0 + tg) * HD + h * D + d, HD, n - tg, d < D, x);
-  load_values(vs, proj + (size_t)t0 * ld + p.cvv + h * E + e0, ld, n, E - e0);
+  load_values<SE>(vs, proj + (size_t)t0 * ld + p.cvv + h * E + e0, ld, n, E - e0, (E & 3) == 0);
   __syncthreads();
   float r = 0.f;
   for (int g = grp + 1; g < NG; g++) r += gsum[g * DP + d];
@@ -113,7 +121,7 @@ __global__ void __launch_bounds__(GC_THREADS) gla_state_kernel(const __grid_cons
   }
   if (blockIdx.x == 0 && grp == 0 && d < D) decay[((size_t)ch * p.H + h) * D + d] = expf(-r);
   __syncthreads();
-  const int m0 = DP >= 128 ? warp * MT : warp & 3, n0 = DP >= 128 ? 0 : (warp >> 2) * 32;
+  const int m0 = DP >= 128 ? warp * MT : warp & 3, n0 = DP >= 128 ? 0 : (warp >> 2) * (SE / 2);
   float u[MT][2 * NT][4];
 #pragma unroll
   for (int i = 0; i < MT; i++)
@@ -129,7 +137,7 @@ __global__ void __launch_bounds__(GC_THREADS) gla_state_kernel(const __grid_cons
 #pragma unroll
     for (int j = 0; j < NT; j++) {
       uint32_t b[4];
-      rc_ldmt(b, rc_bk(vs, GC_ELD, k, n0 + j * 16, lane));
+      rc_ldmt(b, rc_bk(vs, SLD, k, n0 + j * 16, lane));
 #pragma unroll
       for (int i = 0; i < MT; i++)
 #pragma unroll
@@ -160,30 +168,38 @@ __global__ void __launch_bounds__(GC_THREADS) gla_state_kernel(const __grid_cons
 
 // ---- the state down the chunks ------------------------------------------------------------------------
 constexpr int GA_BATCH = 8;
+__device__ __forceinline__ float fma_state(float s, float g, float u) { return fmaf(s, g, u); }
+__device__ __forceinline__ float4 fma_state(float4 s, float g, float4 u) {
+  return make_float4(fmaf(s.x, g, u.x), fmaf(s.y, g, u.y), fmaf(s.z, g, u.z), fmaf(s.w, g, u.w));
+}
+template <typename V>   // float4 where four elements share a row of the state
 __global__ void __launch_bounds__(256) gla_carry_kernel(const __grid_constant__ RecurP p, float* __restrict__ U,
                                                         const float* __restrict__ decay, int chunks, int pos0) {
   pdl_wait();
   pdl_launch_dependents();
-  const int i = blockIdx.x * 256 + threadIdx.x, n = p.H * p.D * p.E;
+  constexpr int W = sizeof(V) / 4;
+  const int i = (blockIdx.x * 256 + threadIdx.x) * W, n = p.H * p.D * p.E;
   if (i >= n) return;
   const int hd = i / p.E, HD = p.H * p.D;
-  float s = pos0 > 0 ? p.S[i] : 0.f;
+  V s{};
+  if (pos0 > 0) s = *(const V*)(p.S + i);
   for (int c0 = 0; c0 < chunks; c0 += GA_BATCH) {
-    float u[GA_BATCH], g[GA_BATCH];
+    V u[GA_BATCH];
+    float g[GA_BATCH];
 #pragma unroll
     for (int c = 0; c < GA_BATCH; c++)
       if (c0 + c < chunks) {
-        u[c] = U[(size_t)(c0 + c) * n + i];
+        u[c] = *(const V*)(U + (size_t)(c0 + c) * n + i);
         g[c] = decay[(size_t)(c0 + c) * HD + hd];
       }
 #pragma unroll
     for (int c = 0; c < GA_BATCH; c++)
       if (c0 + c < chunks) {
-        U[(size_t)(c0 + c) * n + i] = s;
-        s = fmaf(s, g[c], u[c]);
+        *(V*)(U + (size_t)(c0 + c) * n + i) = s;
+        s = fma_state(s, g[c], u[c]);
       }
   }
-  p.S[i] = s;
+  *(V*)(p.S + i) = s;
 }
 
 // ---- the chunk's outputs --------------------------------------------------------------------------------
@@ -231,7 +247,7 @@ __global__ void __launch_bounds__(GC_THREADS, DP <= 128 ? 2 : 1)
       all += gsum[g * DP + d];
     }
     const bool far = __syncthreads_or(all > GC_MOST);
-#pragma unroll 16
+#pragma unroll
     for (int i = 0; i < TG; i++) {
       const bool on = d < D && tg + i < n;
       const float qv = on ? row[(size_t)i * ld + p.cq] * qscale : 0.f, kv = on && !far ? row[(size_t)i * ld + p.ck] : 0.f;
@@ -290,14 +306,20 @@ __global__ void __launch_bounds__(GC_THREADS, DP <= 128 ? 2 : 1)
     const float* S = U + ((size_t)ch * p.H + h) * D * E;
     for (int e0 = 0; e0 < E; e0 += GC_E) {
       __syncthreads();   // keys, or the columns before, are read
-      load_values(vs, proj + (size_t)t0 * ld + p.cvv + h * E + e0, ld, n, E - e0);
-#pragma unroll 4
+      load_values<GC_E>(vs, proj + (size_t)t0 * ld + p.cvv + h * E + e0, ld, n, E - e0, (E & 3) == 0);
+#pragma unroll 8
       for (int i = tid; i < DP * GC_E / 2; i += GC_THREADS) {
         const int r = i / (GC_E / 2), c = (i - r * (GC_E / 2)) * 2;
         const float* at = S + (size_t)r * E + e0 + c;
-        const float a = r < D && e0 + c < E ? at[0] : 0.f, b2 = r < D && e0 + c + 1 < E ? at[1] : 0.f;
+        float2 v = make_float2(0.f, 0.f);
+        if ((E & 1) == 0) {
+          if (r < D && e0 + c < E) v = *(const float2*)at;
+        } else {
+          if (r < D && e0 + c < E) v.x = at[0];
+          if (r < D && e0 + c + 1 < E) v.y = at[1];
+        }
         uint32_t hi, lo;
-        rc_split(a, b2, hi, lo);
+        rc_split(v.x, v.y, hi, lo);
         *(uint32_t*)(ss + r * GC_ELD + c) = hi;
         *(uint32_t*)(ss + (DP + r) * GC_ELD + c) = lo;
       }
@@ -355,15 +377,18 @@ template <int DP>
 int gla_t(const RecurP& p, const float* proj, long long ld, const float* rates, float* U, float* decay, float* o, int rows,
           int pos0, cudaStream_t s) {
   const int chunks = (rows + GC_L - 1) / GC_L;
-  constexpr int sm1 = (2 * GC_L * (DP + 8) + GC_L * GC_ELD) * 2 + GC_THREADS * 4, sm2 = (int)GoSmem<DP>::TOTAL;
+  constexpr int SE = GS_E<DP>;
+  constexpr int sm1 = (2 * GC_L * (DP + 8) + GC_L * (SE + 8)) * 2 + GC_THREADS * 4, sm2 = (int)GoSmem<DP>::TOTAL;
   static std::atomic<unsigned long long> d1{0}, d2{0};
   int rc = ensure_dynamic_smem(gla_state_kernel<DP>, sm1, d1);
   if (!rc) rc = ensure_dynamic_smem(gla_out_kernel<DP>, sm2, d2);
   if (rc) return rc;
-  LaunchCfg l1(dim3((p.E + GC_E - 1) / GC_E, p.H, chunks), dim3(GC_THREADS), sm1, s, pdl_enabled());
+  LaunchCfg l1(dim3((p.E + SE - 1) / SE, p.H, chunks), dim3(GC_THREADS), sm1, s, pdl_enabled());
   TLB_CUDA(cudaLaunchKernelEx(&l1.cfg, gla_state_kernel<DP>, p, proj, ld, rates, U, decay, rows));
-  LaunchCfg l2(dim3((p.H * p.D * p.E + 255) / 256), dim3(256), 0, s, pdl_enabled());
-  TLB_CUDA(cudaLaunchKernelEx(&l2.cfg, gla_carry_kernel, p, U, (const float*)decay, chunks, pos0));
+  const int w = (p.E & 3) == 0 ? 4 : 1;
+  LaunchCfg l2(dim3((p.H * p.D * p.E / w + 255) / 256), dim3(256), 0, s, pdl_enabled());
+  if (w == 4) TLB_CUDA(cudaLaunchKernelEx(&l2.cfg, gla_carry_kernel<float4>, p, U, (const float*)decay, chunks, pos0));
+  else TLB_CUDA(cudaLaunchKernelEx(&l2.cfg, gla_carry_kernel<float>, p, U, (const float*)decay, chunks, pos0));
   LaunchCfg l3(dim3(p.H, chunks), dim3(GC_THREADS), sm2, s, pdl_enabled());
   TLB_CUDA(cudaLaunchKernelEx(&l3.cfg, gla_out_kernel<DP>, p, proj, ld, rates, (const float*)U, o, rows));
   return TLB_OK;

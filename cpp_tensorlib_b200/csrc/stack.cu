@@ -429,7 +429,7 @@ static int build_latents(StackDecoder* d, DeviceCtx* c) {
     }
     const int units = (p.H + 15) / 16, tiles = (p.window + 63) / 64;
     p.splits = max_i(1, c->sm_count / units);
-    if (p.splits > 32) p.splits = 32;
+    if (p.splits > 64) p.splits = 64;
     if (p.splits > tiles) p.splits = tiles;
     const size_t f = latent_part_floats(p, 1, p.splits), a = (size_t)p.H * p.row() * d->es(), q = (size_t)p.H * p.qw();
     part = f > part ? f : part;
@@ -503,7 +503,7 @@ static int build(StackDecoder* d, const tlb_stack_cfg* cfg, const tlb_layer_cfg*
         d->q_max = max_i(d->q_max, H * p.Dp);
       } else if (k.kind == TLB_MIX_LATENT) {
         TLB_REQUIRE(!L.has_latent, "tlb_stack_create: one latent attention a layer");
-        TLB_REQUIRE(k.q_rank > 0 && k.kv_rank > 0 && k.kv_rank <= 512 && D <= 1024, "tlb_stack_create: latent too wide");
+        TLB_REQUIRE(k.q_rank > 0 && k.kv_rank > 0 && k.kv_rank <= 8192 && D <= 1024, "tlb_stack_create: latent too wide");
         TLB_REQUIRE(k.window >= 0 && k.rot_dims >= 0 && k.rot_dims <= 2 * MX_PAIRS && k.rot_dims % 2 == 0,
                     "tlb_stack_create: bad window or rotation");
         L.has_latent = true;

@@ -40,13 +40,15 @@ CONFIGS = dict(
     base=config([full(), gla(), win(), full(kv_from=0, heads=2, vdim=24), gla(ff=0), win(ff=0, heads=8)]),
     # nothing a multiple of anything, one head, decays of every strength
     odd=config([gla(3, 9, 7, 1.0, 37), win(7, 3, 11, 6, 13, 21, 19, ff=0), full(1, 5, 2, 3, 7, 10, ff=11), gla(1, 21, 13, 3.0, 0),
-                full(5, 10, 2, 6, 9, 10, kv_from=2)], width=52, vocab=71, logit_scale=0.3),
+                full(5, 10, 2, 6, 9, 10, kv_from=2)], width=45, vocab=71, logit_scale=0.3),
     # more heads than a tile of 16, a latent and heads that the prompt tiles do not take, a state too wide for chunks
     wide=config([full(20, 144, 56, 24, 40, 200, ff=56), gla(2, 264, 40, 16.0), win(4000, 17, 24, 8, 136, 33, 136),
                  full(18, 8, 56, 16, 40, 200, kv_from=0)], width=72, vocab=128),
     # the widths the tiled kernels are made for
     real=config([win(150, 8, 128, 64, 128, 96, 512, ff=192), gla(2, 128, 128, 16.0), full(4, 64, 32, 64, 64, 256, ff=128),
                  gla(3, 64, 192, 8.0), full(2, 96, 32, 96, 72, 256, kv_from=2), gla(1, 200, 72, 4.0)], width=128, vocab=160),
+    # a latent wider than the tensor-pipe decoding takes, more than one pass of its columns
+    deep=config([full(5, 16, 8, 24, 40, 1064), gla(3, 20, 28), full(2, 192, 8, 8, 16, 1064, kv_from=0)], vocab=88),
     narrow=config([gla(2, 48, 32, 5.0, 64), full(2, 8, 56, 32, 16, 64), win(33, 6, 40, 8, 48, 24, 120)], width=96, vocab=64),
 )
 

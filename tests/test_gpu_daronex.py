@@ -426,6 +426,6 @@ def test_refusals():
     close(m)
     for bad in (dc.config([dc.full(kv_from=0)]), dc.config([dc.full(), dc.full(kv_rank=40, kv_from=0)]),
                 dc.config([dc.gla(), dc.full(kv_from=0)]), dc.config([dc.full(), dc.full(kv_from=0), dc.full(kv_from=1)]),
-                dc.config([dc.full(kv_rank=520)])):
+                dc.config([dc.full(kv_rank=9000)])):
         with pytest.raises(TlbError):
             make(bad, weights(bad, 1), "bfloat16", 32)
